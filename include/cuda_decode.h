@@ -116,6 +116,9 @@ const char* cd_last_error(const cd_model* m);
 /* Model::len / Model::set_len (clamped to seq), lib.rs:209-215. */
 int cd_len(const cd_model* m, size_t* len);
 int cd_set_len(cd_model* m, size_t len);
+/* 1 when cd_set_len(m, len) would succeed.  A family with recurrent state (the configured decoders below) keeps that
+ * state at the ends of the last few cd_prefill calls; it can go back to one of those lengths, or to 0. */
+int cd_can_rewind(const cd_model* m, size_t len);
 
 /* Model::seed_layer_cache_from_channel_first, lib.rs:217-237: k_rope_cf and v_cf
  * are [kv_dim, seq] channel-first fp32; rows >= live_len are zeroed. */
@@ -215,6 +218,21 @@ int cd_moe_shard_plan(const cd_config* cfg, const cd_moe_config* moe, int world,
 /* the experts the router chose in `layer` at the last decoded position, best first (top_k ids) */
 int cd_moe_last_experts(cd_model* m, int layer, int32_t* out_ids, size_t cap);
 
+/* ---------------------------------------------------------------- additive: configured decoders
+ * A model folder holds config.json, whose "architecture" names an entry of the library's registry, and
+ * model.safetensors (no counterpart in the reference, whose one architecture is fixed by its checkpoint header).
+ * Registered: "Dafidra" - per layer a windowed softmax attention (whole-projection q/k norm, query temperature, linear
+ * distance bias, sink, per-head output gate) and a matrix memory (mLSTM) side by side on the un-normed residual stream,
+ * norms on the sublayers' outputs, then a dense or a routed feed-forward.
+ * opts->weight_dtype: CD_DTYPE_BF16 (also for < 0) or CD_DTYPE_F32; one GPU.  max_tokens (0: 4096) bounds the sequence:
+ * it becomes cd_config.seq.  Every call that takes a cd_model works on the handle except cd_seed_layer_cache_cf and
+ * cd_decode_steps_samples (CD_ERR_UNSUPPORTED; the session then runs the samples one after the other).
+ * cd_model_create_from_config: the same with seeded synthetic matrices ~N(0, std), norms 1, for a configuration given
+ * as JSON text.  cd_config_info parses and validates such a text on the host (no GPU); seq is 0 in its result. */
+int cd_model_create_from_dir(const char* dir, size_t max_tokens, const cd_options* opts, cd_model** out);
+int cd_model_create_from_config(const char* config_json, size_t max_tokens, const cd_options* opts, uint64_t seed, float std, cd_model** out);
+int cd_config_info(const char* config_json, cd_config* cfg_out);
+
 /* ---------------------------------------------------------------- additive: tensor parallelism
  * One process per GPU.  Create each rank's model with opts->tp_world = world size (2, 4 or 8)
  * and opts->tp_rank = rank: it keeps heads/world attention heads, hidden/world FFN columns
@@ -250,11 +268,14 @@ int cd_decode_token_logits_from_id(cd_model* m, uint32_t token, float softcap, f
 /* Prefill n prompt tokens starting at the current len; last_logits (optional,
  * [vocab]) receives the logits of the last prompt position — what
  * InferenceSession::new (inference.rs:124-161) keeps of its forward pass.  With n >= 8 on a
- * bf16 / fp16 / FP8 single-GPU model the tokens are processed together (tensor-core GEMMs,
+ * bf16 / fp16 / FP8 single-GPU model (dense or configured) the tokens are processed together (tensor-core GEMMs,
  * K and V written into the decode pages); otherwise one at a time as
  * prefill_prompt_suffix_cached does (inference.rs:650-670).  The first batched call
  * allocates a workspace that grows with the longest prompt seen. */
 int cd_prefill(cd_model* m, const uint32_t* ids, size_t n, float softcap, float* last_logits);
+/* The same with logits at chosen places: row k of out ([nwant][vocab]) is the logits after token want[k] (0 .. n-1) of
+ * this call. */
+int cd_prefill_logits(cd_model* m, const uint32_t* ids, size_t n, const size_t* want, size_t nwant, float softcap, float* out);
 
 /* run_cached_sample's three hot loops (inference.rs:576-625) without a host round
  * trip per token: feed first_token, produce nsteps further tokens.  Only token

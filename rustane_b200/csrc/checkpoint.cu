@@ -186,7 +186,7 @@ int cd_model_create_from_checkpoint(const char* path, const cd_options* opts_in,
     }
     opts.activation = (int)h.activation;
     cd_model* m = nullptr;
-    rc = model_alloc(&h.cfg, &opts, (int)h.untied, &m);
+    rc = dense_alloc(&h.cfg, &opts, (int)h.untied, &m);
     if (rc) { fclose(f); return rc; }
 
     std::vector<uint8_t> raw;
@@ -274,7 +274,7 @@ int cd_model_save_quantised(cd_model* m, const char* path) {
     if (!m || !path) return fail(m, CD_ERR_INVALID, "null argument");
     const int dt = m->opt.weight_dtype;
     if (dt != CD_DTYPE_FP8_E4M3 && dt != CD_DTYPE_INT4_G32) return fail(m, CD_ERR_INVALID, "the model's linears are not quantised");
-    if (m->tp_world > 1 || m->moe) return fail(m, CD_ERR_UNSUPPORTED, "a quantised checkpoint is written from a whole dense model (one GPU)");
+    if (m->tp_world > 1) return fail(m, CD_ERR_UNSUPPORTED, "a quantised checkpoint is written from a whole dense model (one GPU)");
     const cd_config& c = m->full_cfg;
     FILE* f = fopen(path, "wb");
     if (!f) return fail(m, CD_ERR_IO, std::string("cannot create ") + path);

@@ -117,14 +117,21 @@ struct EpiGateMoe {
 // SrcPlain: one matrix, row r at W + r * row_bytes.  The two expert sources assemble a virtual matrix from
 // the experts the router chose for this token (a device-side list, so the kernel reads its shape after
 // waiting for the previous kernel): the producer's copies gather it, the consumers see plain rows.
-constexpr int SRC_MAX_LIST = 16;  // entries of a chosen-expert list (top_k at most)
+constexpr int SRC_MAX_LIST = 32;  // entries of a chosen-expert list (top_k at most)
 struct SrcPlain {
-    static constexpr bool DYNAMIC = false;
+    static constexpr bool DYNAMIC = false, PAIR = false;
+};
+// Two matrices in one launch: CTAs 0 .. split-1 stream the first, the rest the second (its own input width); the
+// second one's outputs are numbered behind the first one's.  The CTAs are split by bytes, so both end together.
+struct SrcPair {
+    static constexpr bool DYNAMIC = false, PAIR = true;
+    const void* w2;
+    int n2, k2, split;
 };
 // Rows in blocks: entry s of the list contributes seg_rows rows (expert list[s] of W), then tail_rows rows of `tail`.
 // `list` is the CTA's shared-memory copy of loc_ids, nl its length.
 struct SrcExpertRows {
-    static constexpr bool DYNAMIC = true;
+    static constexpr bool DYNAMIC = true, PAIR = false;
     const int* loc_ids;
     const int* n_loc;
     const void* tail;
@@ -148,7 +155,7 @@ struct SrcExpertRows {
 // Columns in blocks: row r is the concatenation of row r of expert list[s] (seg_bytes each, the expert's matrix has
 // mat_rows rows) for every list entry, then row r of `tail` (tail_bytes).
 struct SrcExpertCols {
-    static constexpr bool DYNAMIC = true;
+    static constexpr bool DYNAMIC = true, PAIR = false;
     const int* loc_ids;
     const int* n_loc;
     const void* tail;
@@ -196,12 +203,30 @@ __device__ inline float consumer_sum(float v, float* red, int group = 0) {  // r
     return t;
 }
 
-template <typename WT, int NITER, int R, int UNIT, bool NORM, class Epi, int G = 1, class Src = SrcPlain>
+// How the input vector comes about.  GemvIn: the vector x, under NORM divided by its root mean square and times gamma,
+// or under tensor parallelism res + alpha * (sum of the ranks' partial vectors).  Other input types (CUSTOM) fill the
+// consumers' registers themselves: load(registers, thread, chunks, 8 floats of shared memory, group, whether the CTA
+// works on the second matrix of a pair, whether this thread's copy is the one to publish).
+struct GemvIn {
+    static constexpr bool CUSTOM = false;
+};
+
+template <typename WT, int NITER, int R, int UNIT, bool NORM, class Epi, int G = 1, class Src = SrcPlain, class In = GemvIn>
 __global__ void __launch_bounds__(G * GEMV_CONSUMERS + 32, 1)
 gemv_tma_kernel(const WT* __restrict__ W, const float* __restrict__ x, const float* __restrict__ gamma,
                 float* __restrict__ norm_out, int N, int K, int rows_cap, int nstages, int* err, NextStream next,
-                TpLink tp, Epi epi, Src src) {
+                TpLink tp, Epi epi, Src src, float eps, In in) {
     using F = Wfmt<WT>;
+    int bid = blockIdx.x, nblk = gridDim.x, unit0 = 0;
+    if constexpr (Src::PAIR) {
+        if (bid >= src.split) {
+            unit0 = N / UNIT;
+            W = reinterpret_cast<const WT*>(src.w2); N = src.n2; K = src.k2;
+            bid -= src.split; nblk -= src.split;
+        } else {
+            nblk = src.split;
+        }
+    }
     __shared__ int src_list[SRC_MAX_LIST];
     int src_n = 0;
     if constexpr (Src::DYNAMIC) {  // the shape is the previous kernel's result; N and K arrive as its upper bounds
@@ -231,8 +256,8 @@ gemv_tma_kernel(const WT* __restrict__ W, const float* __restrict__ x, const flo
     const int gwarp = G == 1 ? warp : (warp & (NW - 1));
     const int nchunks = K / EPC;
     const int nunits = N / UNIT;
-    const int u0 = (int)((long long)blockIdx.x * nunits / gridDim.x);
-    const int u1 = (int)((long long)(blockIdx.x + 1) * nunits / gridDim.x);
+    const int u0 = (int)((long long)bid * nunits / nblk);
+    const int u1 = (int)((long long)(bid + 1) * nunits / nblk);
     const int r0 = u0 * UNIT, r1 = u1 * UNIT;
     const int ngroups = K > 0 ? (r1 - r0 + R - 1) / R : 0;  // K == 0 (an empty expert list and no tail): every output is zero
 
@@ -278,6 +303,9 @@ gemv_tma_kernel(const WT* __restrict__ W, const float* __restrict__ x, const flo
     pdl_wait();
     pdl_launch_dependents();  // after the wait: at most this kernel and the next one overlap
     float xr[NITER][EPC];
+    if constexpr (In::CUSTOM) {
+        in.load(xr, tid, nchunks, red + 8 * group, group, Src::PAIR && unit0 > 0, bid == 0 && unit0 == 0 && group == 0);
+    } else {
     float ss = 0.0f;
     const float* inbox = nullptr;  // tensor parallel: the input is res + alpha * (sum of the peers' partial vectors)
     if (tp.world > 1 && tp.in_reduce) {
@@ -313,7 +341,7 @@ gemv_tma_kernel(const WT* __restrict__ W, const float* __restrict__ x, const flo
     }
     if (NORM) {
         const float tot = consumer_sum(ss, red + 8 * group, group);
-        const float inv = 1.0f / sqrtf(tot * (1.0f / (float)K) + RMS_EPS);
+        const float inv = 1.0f / sqrtf(tot * (1.0f / (float)K) + eps);
 #pragma unroll
         for (int i = 0; i < NITER; ++i) {
             const int c = tid + i * GEMV_CONSUMERS;
@@ -331,6 +359,7 @@ gemv_tma_kernel(const WT* __restrict__ W, const float* __restrict__ x, const flo
                 }
             }
         }
+    }
     }
 
     bool ok = true;
@@ -398,7 +427,7 @@ gemv_tma_kernel(const WT* __restrict__ W, const float* __restrict__ x, const flo
             for (int wi = 0; wi < NW; ++wi) sacc += partial[(u * UNIT + k) * NW + wi];
             y[k] = ngroups > 0 ? sacc : 0.0f;
         }
-        epi(u0 + u, y);
+        epi(unit0 + u0 + u, y);
     }
 }
 

@@ -1,0 +1,494 @@
+// Token mixers and vector pre-steps of the configured decoder (hybrid.h), one token per step.  Each mechanism takes its
+// sizes and constants as parameters:
+//   windowed softmax attention   whole-projection RMS norm of q and k, a temperature on q that grows with the position,
+//                                a linear distance bias per head, a sink in the denominator, one output gate per head,
+//                                key and value widths of their own, paged cache
+//   matrix memory (mLSTM)        S <- f S + i k v^T per head with exponential input gate, sigmoid forget gate and a running
+//                                maximum; fp32 state in HBM, updated in place
+//   GEMV inputs                  residual + norm of a sublayer's output, the average of two normed outputs, and the
+//                                memory's per-head norm and gate, folded into the GEMV that consumes the vector
+// Both mixers of a layer run in one launch (mixer_step_kernel).  The routing rule shared by the decode router and the
+// batched one is route_pick (moe.cuh).
+#pragma once
+#include "common.cuh"
+#include "kernels.cuh"
+
+namespace cd {
+
+// Offsets of the projections in one row of proj [rows]: left (attention) q | k | v | gate, right (memory)
+// q | k | v | gate | input gate | forget gate.
+struct ProjLayout {
+    int lq, lk, lv, lg, rq, rk, rv, rg, ri, rf, rows;
+};
+
+struct AttnDims {
+    int H, G, dim, vdim;
+    int kp, vp;          // key / value row widths in the cache: dim and vdim padded to 16 with zeros
+    int window;          // positions seen, itself included; 0: all
+    int page_tokens;
+    float scale, eps, temp_coef;
+    int temp_every;
+    // a page: K [G][page_tokens][kp], then V [G][page_tokens][vp]
+    __host__ __device__ size_t page_elems() const { return (size_t)G * page_tokens * (kp + vp); }
+    __host__ __device__ size_t k_at(int page, int g, int off) const { return (size_t)page * page_elems() + ((size_t)g * page_tokens + off) * kp; }
+    __host__ __device__ size_t v_at(int page, int g, int off) const {
+        return (size_t)page * page_elems() + (size_t)G * page_tokens * kp + ((size_t)g * page_tokens + off) * vp;
+    }
+    __device__ float temperature(int pos) const {
+        return temp_coef == 0.0f ? 1.0f : 1.0f + temp_coef * logf((float)((pos + 1) / temp_every) + 1.0f);
+    }
+};
+
+// State of one layer: S [H][dim][vs], n [H][nslice][dim], m [H][nslice].  A slice of MEM_SLICE value columns of a head is
+// one CTA's work; n and m are kept once per slice (each CTA updates its own copy, so no CTA waits for another).
+constexpr int MEM_SLICE = 32;
+struct MemDims {
+    int H, dim, vdim;
+    int vs;              // row stride of S: vdim padded to 4
+    int nslice;          // ceil(vdim / MEM_SLICE)
+    float cap, eps;
+    __host__ __device__ size_t s_floats() const { return (size_t)H * dim * vs; }
+    __host__ __device__ size_t n_off() const { return s_floats(); }
+    __host__ __device__ size_t m_off() const { return s_floats() + (size_t)H * nslice * dim; }
+    __host__ __device__ size_t floats() const { return (m_off() + (size_t)H * nslice + 63) / 64 * 64; }
+};
+
+__device__ inline float soft_cap(float z, float cap) { return cap * tanhf(z / cap); }
+__device__ inline float log_sigmoid(float z) { return fminf(z, 0.0f) - log1pf(expf(-fabsf(z))); }
+__device__ inline float sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+// ---------------------------------------------------------------------- inputs of the streamed GEMV (kernels.cuh, GemvIn)
+// x' = x + mult * gain * y / rms(y): the residual stream after a sublayer whose output is normed
+struct InNormedResidual {
+    static constexpr bool CUSTOM = true;
+    const float *x, *y, *gain;
+    float* x_out;
+    float mult, eps;
+    int n;
+    template <int NITER, int EPC>
+    __device__ void load(float (&xr)[NITER][EPC], int tid, int nchunks, float* red, int group, bool, bool writer) const {
+        float ss = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NITER; ++i) {
+            const int c = tid + i * GEMV_CONSUMERS;
+#pragma unroll
+            for (int e = 0; e < EPC; e += 4) {
+                float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (c < nchunks) v = __ldcg(reinterpret_cast<const float4*>(y + (size_t)c * EPC + e));
+                xr[i][e] = v.x; xr[i][e + 1] = v.y; xr[i][e + 2] = v.z; xr[i][e + 3] = v.w;
+                ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+            }
+        }
+        const float r = mult / sqrtf(consumer_sum(ss, red, group) * (1.0f / (float)n) + eps);
+#pragma unroll
+        for (int i = 0; i < NITER; ++i) {
+            const int c = tid + i * GEMV_CONSUMERS;
+            if (c >= nchunks) continue;
+#pragma unroll
+            for (int e = 0; e < EPC; e += 4) {
+                const float4 b = __ldcg(reinterpret_cast<const float4*>(x + (size_t)c * EPC + e)), g = *reinterpret_cast<const float4*>(gain + (size_t)c * EPC + e);
+                xr[i][e] = b.x + xr[i][e] * r * g.x; xr[i][e + 1] = b.y + xr[i][e + 1] * r * g.y;
+                xr[i][e + 2] = b.z + xr[i][e + 2] * r * g.z; xr[i][e + 3] = b.w + xr[i][e + 3] * r * g.w;
+                if (writer) *reinterpret_cast<float4*>(x_out + (size_t)c * EPC + e) = make_float4(xr[i][e], xr[i][e + 1], xr[i][e + 2], xr[i][e + 3]);
+            }
+        }
+    }
+};
+
+// x' = x + mult * gain * z / rms(z),  z = (wl * yl / rms(yl) + wr * yr / rms(yr)) / 2: the same behind two parallel mixers
+struct InParallelMix {
+    static constexpr bool CUSTOM = true;
+    const float *x, *yl, *yr, *wl, *wr, *gain;
+    float* x_out;
+    float mult, eps;
+    int n;
+    template <int NITER, int EPC>
+    __device__ void load(float (&xr)[NITER][EPC], int tid, int nchunks, float* red, int group, bool, bool writer) const {
+        float sl = 0.0f, sr = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NITER; ++i) {
+            const int c = tid + i * GEMV_CONSUMERS;
+#pragma unroll
+            for (int e = 0; e < EPC; e += 4) {
+                if (c < nchunks) {
+                    const float4 a = __ldcg(reinterpret_cast<const float4*>(yl + (size_t)c * EPC + e)), b = __ldcg(reinterpret_cast<const float4*>(yr + (size_t)c * EPC + e));
+                    sl += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+                    sr += b.x * b.x + b.y * b.y + b.z * b.z + b.w * b.w;
+                }
+            }
+        }
+        const float rl = 0.5f / sqrtf(consumer_sum(sl, red, group) * (1.0f / (float)n) + eps);
+        const float rr = 0.5f / sqrtf(consumer_sum(sr, red, group) * (1.0f / (float)n) + eps);
+        float ss = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NITER; ++i) {
+            const int c = tid + i * GEMV_CONSUMERS;
+#pragma unroll
+            for (int e = 0; e < EPC; e += 4) {
+                float4 z = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (c < nchunks) {
+                    const size_t at = (size_t)c * EPC + e;
+                    const float4 a = __ldcg(reinterpret_cast<const float4*>(yl + at)), b = __ldcg(reinterpret_cast<const float4*>(yr + at));
+                    const float4 p = *reinterpret_cast<const float4*>(wl + at), q = *reinterpret_cast<const float4*>(wr + at);
+                    z = make_float4(a.x * rl * p.x + b.x * rr * q.x, a.y * rl * p.y + b.y * rr * q.y, a.z * rl * p.z + b.z * rr * q.z, a.w * rl * p.w + b.w * rr * q.w);
+                }
+                xr[i][e] = z.x; xr[i][e + 1] = z.y; xr[i][e + 2] = z.z; xr[i][e + 3] = z.w;
+                ss += z.x * z.x + z.y * z.y + z.z * z.z + z.w * z.w;
+            }
+        }
+        const float r = mult / sqrtf(consumer_sum(ss, red, group) * (1.0f / (float)n) + eps);
+#pragma unroll
+        for (int i = 0; i < NITER; ++i) {
+            const int c = tid + i * GEMV_CONSUMERS;
+            if (c >= nchunks) continue;
+#pragma unroll
+            for (int e = 0; e < EPC; e += 4) {
+                const size_t at = (size_t)c * EPC + e;
+                const float4 b = __ldcg(reinterpret_cast<const float4*>(x + at)), g = *reinterpret_cast<const float4*>(gain + at);
+                xr[i][e] = b.x + xr[i][e] * r * g.x; xr[i][e + 1] = b.y + xr[i][e + 1] * r * g.y;
+                xr[i][e + 2] = b.z + xr[i][e + 2] * r * g.z; xr[i][e + 3] = b.w + xr[i][e + 3] * r * g.w;
+                if (writer) *reinterpret_cast<float4*>(x_out + at) = make_float4(xr[i][e], xr[i][e + 1], xr[i][e + 2], xr[i][e + 3]);
+            }
+        }
+    }
+};
+
+// Input of the paired output projections: the first matrix takes the gated attention output as it is; the second takes
+// the memory's raw read-out, each head divided by its root mean square (the sums of squares arrive per slice), times
+// the norm weight, times the sigmoid of the gate projection.
+struct InMixerOutputs {
+    static constexpr bool CUSTOM = true;
+    const float *attn, *mem, *ssq, *norm, *gate;
+    int n, vdim, nslice;
+    float eps;
+    template <int NITER, int EPC>
+    __device__ void load(float (&xr)[NITER][EPC], int tid, int nchunks, float*, int, bool second, bool) const {
+        int hcur = -1;
+        float rstd = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NITER; ++i) {
+            const int c = tid + i * GEMV_CONSUMERS;
+#pragma unroll
+            for (int e = 0; e < EPC; e += 4) {
+                float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (c < nchunks) v = __ldcg(reinterpret_cast<const float4*>((second ? mem : attn) + (size_t)c * EPC + e));
+                xr[i][e] = v.x; xr[i][e + 1] = v.y; xr[i][e + 2] = v.z; xr[i][e + 3] = v.w;
+            }
+            if (second && c < nchunks) {
+#pragma unroll
+                for (int e = 0; e < EPC; ++e) {
+                    const int j = c * EPC + e;
+                    if (j < n) {
+                        const int h = j / vdim;
+                        if (h != hcur) {
+                            float s = 0.0f;
+                            for (int k = 0; k < nslice; ++k) s += __ldcg(ssq + h * nslice + k);
+                            rstd = 1.0f / sqrtf(s / (float)vdim + eps);
+                            hcur = h;
+                        }
+                        xr[i][e] = xr[i][e] * rstd * norm[j] * sigmoid(__ldcg(gate + j));
+                    }
+                }
+            }
+        }
+    }
+};
+
+// The residual stream after the last layer as a vector in memory (one CTA); widths up to 16384.
+template <class In>
+__global__ void __launch_bounds__(GEMV_CONSUMERS) vector_input_kernel(In in, int n) {
+    __shared__ float red[32];
+    pdl_wait();
+    pdl_launch_dependents();
+    if (n <= 4 * 4 * GEMV_CONSUMERS) {
+        float xr[4][4];
+        in.load(xr, threadIdx.x, n / 4, red, 0, false, true);
+    } else {
+        float xr[16][4];
+        in.load(xr, threadIdx.x, n / 4, red, 0, false, true);
+    }
+}
+
+// ---------------------------------------------------------------------- one token through both mixers of a layer
+struct MixerStep {
+    AttnDims a;
+    MemDims d;
+    ProjLayout pl;
+    const float* proj;                 // this token's projections
+    const float *q_norm, *k_norm, *sink, *slopes;
+    const float *ib, *fb;
+    const int* page_table;
+    const DevState* st;
+    float *part_acc, *part_ml;         // [H][nsplit][vp], [H][nsplit][2]
+    unsigned int* counters;            // [H]
+    float* attn;                       // [H * vdim], gated
+    float* mem;                        // [Hr * vdim], raw read-out
+    float* ssq;                        // [Hr][nslice]
+    float* state;                      // this layer's state
+    int nsplit;
+};
+constexpr int MIX_THREADS = 128, MIX_TILE = 32;
+__host__ __device__ inline size_t mixer_attn_smem_floats(int kp, int vp) { return (size_t)2 * kp + vp + (size_t)MIX_THREADS * 8 + MIX_TILE + 96; }
+__host__ __device__ inline size_t mixer_mem_smem_floats(int dim) { return (size_t)2 * dim + 4 * MEM_SLICE + 64; }
+
+// A matrix-memory slice: MEM_SLICE value columns of one head.  128 threads = 16 row groups x 8 column quads.
+__device__ inline void mem_step(const MixerStep& p, int idx, float* sm, float* red) {
+    const MemDims& d = p.d;
+    const int h = idx / d.nslice, sl = idx % d.nslice, tid = threadIdx.x;
+    const int rg = tid >> 3, col = sl * MEM_SLICE + (tid & 7) * 4;
+    float* S = p.state + (size_t)h * d.dim * d.vs + col;
+    float* nvec = p.state + d.n_off() + ((size_t)h * d.nslice + sl) * d.dim;
+    float* mrun = p.state + d.m_off() + h * d.nslice + sl;
+    const bool live = col < d.vdim;
+    // this CTA's part of the state was written a whole token ago: its first rows are requested before the previous
+    // kernel of the chain has finished (at most two neighbours of the chain overlap)
+    constexpr int PRE = 8;
+    float4 s[PRE];
+#pragma unroll
+    for (int j = 0; j < PRE; ++j) {
+        const int r = rg + 16 * j;
+        s[j] = live && r < d.dim ? __ldcg(reinterpret_cast<const float4*>(S + (size_t)r * d.vs)) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    pdl_wait();
+    pdl_launch_dependents();
+    float* qs = sm;
+    float* ks = sm + d.dim;
+    float* acc_s = sm + 2 * d.dim;  // [4 warps][MEM_SLICE]
+    const float zi = __ldcg(p.proj + p.pl.ri + h) + p.ib[h], zf = __ldcg(p.proj + p.pl.rf + h) + p.fb[h];
+    const float gi = soft_cap(zi, d.cap), gf = log_sigmoid(soft_cap(zf, d.cap));
+    const float m0 = __ldcg(mrun), mt = fmaxf(gf + m0, gi), fa = expf(gf + m0 - mt), ia = expf(gi - mt);
+    const float qscale = 1.0f / sqrtf((float)d.dim);
+    float nq = 0.0f;
+    for (int i = tid; i < d.dim; i += MIX_THREADS) {
+        const float q = __ldcg(p.proj + p.pl.rq + h * d.dim + i) * qscale, k = __ldcg(p.proj + p.pl.rk + h * d.dim + i);
+        qs[i] = q;
+        ks[i] = k;
+        const float nn = fa * __ldcg(nvec + i) + ia * k;
+        nvec[i] = nn;
+        nq = fmaf(nn, q, nq);
+    }
+    nq = block_sum(nq, red);  // (its barriers publish qs and ks)
+    if (tid == 0) *mrun = mt;
+    float v[4], acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[e] = col + e < d.vdim ? ia * __ldcg(p.proj + p.pl.rv + h * d.vdim + col + e) : 0.0f;
+    for (int r0 = rg; r0 < d.dim; r0 += 16 * PRE) {
+        if (r0 != rg) {
+#pragma unroll
+            for (int j = 0; j < PRE; ++j) {
+                const int r = r0 + 16 * j;
+                s[j] = live && r < d.dim ? __ldcg(reinterpret_cast<const float4*>(S + (size_t)r * d.vs)) : make_float4(0.f, 0.f, 0.f, 0.f);
+            }
+        }
+#pragma unroll
+        for (int j = 0; j < PRE; ++j) {
+            const int r = r0 + 16 * j;
+            if (r < d.dim) {
+                const float k = ks[r], q = qs[r];
+                const float4 t = make_float4(fmaf(fa, s[j].x, k * v[0]), fmaf(fa, s[j].y, k * v[1]), fmaf(fa, s[j].z, k * v[2]), fmaf(fa, s[j].w, k * v[3]));
+                if (live) *reinterpret_cast<float4*>(S + (size_t)r * d.vs) = t;
+                acc[0] = fmaf(q, t.x, acc[0]); acc[1] = fmaf(q, t.y, acc[1]); acc[2] = fmaf(q, t.z, acc[2]); acc[3] = fmaf(q, t.w, acc[3]);
+            }
+        }
+    }
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+        acc[e] += __shfl_xor_sync(0xffffffffu, acc[e], 8);
+        acc[e] += __shfl_xor_sync(0xffffffffu, acc[e], 16);
+    }
+    if ((tid & 31) < 8) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) acc_s[(tid >> 5) * MEM_SLICE + (tid & 7) * 4 + e] = acc[e];
+    }
+    __syncthreads();
+    if (tid < MEM_SLICE) {
+        const int c = sl * MEM_SLICE + tid;
+        const float num = acc_s[tid] + acc_s[MEM_SLICE + tid] + acc_s[2 * MEM_SLICE + tid] + acc_s[3 * MEM_SLICE + tid];
+        const float o = num / (fmaxf(fabsf(nq), expf(-mt)) + 1e-6f);
+        if (c < d.vdim) p.mem[h * d.vdim + c] = o;
+        const float ss = warp_sum(c < d.vdim ? o * o : 0.0f);
+        if (tid == 0) p.ssq[h * d.nslice + sl] = ss;
+    }
+}
+
+// One head's slice of the window: scores of MIX_TILE positions at a time, running softmax, weighted values; slices are
+// merged by the CTA of the head that arrives last (a counter, nobody waits), which adds the sink and the head's gate.
+template <typename KT>
+__device__ inline void attn_step(const MixerStep& p, KT* __restrict__ pool, int idx, float* sm, float* red, int& s_last) {
+    constexpr int EPC = Elem<KT>::EPC;
+    constexpr float NEG = -3.402823466e+38f;
+    const AttnDims& a = p.a;
+    const int h = idx / p.nsplit, sl = idx % p.nsplit, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int gqa = a.H / a.G, g = h / gqa;
+    float* qs = sm;                       // [kp] normed query, temperature and scale folded in
+    float* kc = qs + a.kp;                // [kp] this position's key as the cache holds it
+    float* vc = kc + a.kp;                // [vp]
+    float* accs = vc + a.vp;              // [128 threads][8]
+    float* ps = accs + MIX_THREADS * 8;   // [MIX_TILE]
+    pdl_wait();
+    pdl_launch_dependents();
+    const int pos = __ldcg(&p.st->pos);
+    const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0, len = pos + 1 - lo;
+    int per = (len + p.nsplit - 1) / p.nsplit;
+    per = (per + MIX_TILE - 1) / MIX_TILE * MIX_TILE;
+    const int t0 = lo + sl * per, t1 = min(pos + 1, t0 + per);
+    float m = NEG, l = 0.0f, acc[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) acc[e] = 0.0f;
+    const int nvc = a.vp / EPC;           // value chunks of a row
+    int lv = 1;
+    while (lv < nvc) lv <<= 1;            // lanes that share a row of values
+    const int vch = tid % lv, vgrp = tid / lv, vgroups = MIX_THREADS / lv;
+    if (t0 < t1) {
+        float sq = 0.0f, sk = 0.0f;
+        const bool newest = t1 == pos + 1;  // this slice holds the current position
+        for (int i = tid; i < a.H * a.dim; i += MIX_THREADS) { const float v = __ldcg(p.proj + p.pl.lq + i); sq = fmaf(v, v, sq); }
+        if (newest)
+            for (int i = tid; i < a.G * a.dim; i += MIX_THREADS) { const float v = __ldcg(p.proj + p.pl.lk + i); sk = fmaf(v, v, sk); }
+        const float rq = a.temperature(pos) * a.scale / sqrtf(block_sum(sq, red) / (float)(a.H * a.dim) + a.eps);
+        for (int i = tid; i < a.kp; i += MIX_THREADS)
+            qs[i] = i < a.dim ? __ldcg(p.proj + p.pl.lq + h * a.dim + i) * rq * p.q_norm[h * a.dim + i] : 0.0f;
+        if (newest) {
+            const float rk = 1.0f / sqrtf(block_sum(sk, red) / (float)(a.G * a.dim) + a.eps);
+            const int page = p.page_table[pos / a.page_tokens], off = pos % a.page_tokens;
+            const bool writer = h % gqa == 0;
+            for (int i = tid; i < a.kp; i += MIX_THREADS) {
+                const KT v = Elem<KT>::from_f32(i < a.dim ? __ldcg(p.proj + p.pl.lk + g * a.dim + i) * rk * p.k_norm[g * a.dim + i] : 0.0f);
+                kc[i] = Elem<KT>::to_f32(v);
+                if (writer) pool[a.k_at(page, g, off) + i] = v;
+            }
+            for (int i = tid; i < a.vp; i += MIX_THREADS) {
+                const KT v = Elem<KT>::from_f32(i < a.vdim ? __ldcg(p.proj + p.pl.lv + g * a.vdim + i) : 0.0f);
+                vc[i] = Elem<KT>::to_f32(v);
+                if (writer) pool[a.v_at(page, g, off) + i] = v;
+            }
+        }
+        __syncthreads();
+        const int nkc = a.kp / EPC;
+        int lk = 1;
+        while (lk < nkc && lk < 32) lk <<= 1;  // lanes that share a key row
+        const int kch = lane % lk, side = 32 / lk;
+        const float slope = p.slopes[h];
+        for (int tb = t0; tb < t1; tb += MIX_TILE) {
+            // scores: warp w takes positions tb + 8 w .. + 7
+            for (int j0 = 0; j0 < 8; j0 += 4 * side) {
+                float d[4] = {0.f, 0.f, 0.f, 0.f};
+                for (int c = kch; c < nkc; c += lk) {
+                    uint4 w[4];
+#pragma unroll
+                    for (int u = 0; u < 4; ++u) {
+                        const int j = j0 + u * side + lane / lk, t = tb + 8 * warp + j;
+                        w[u] = make_uint4(0, 0, 0, 0);
+                        if (j < 8 && t < t1 && t != pos) {
+                            const int page = p.page_table[t / a.page_tokens];
+                            w[u] = ldg_stream_coherent(pool + a.k_at(page, g, t % a.page_tokens) + (size_t)c * EPC);
+                        }
+                    }
+#pragma unroll
+                    for (int u = 0; u < 4; ++u) {
+                        const int j = j0 + u * side + lane / lk, t = tb + 8 * warp + j;
+                        float f[EPC];
+                        Elem<KT>::unpack(w[u], f);
+                        if (t == pos) {
+#pragma unroll
+                            for (int e = 0; e < EPC; ++e) f[e] = kc[c * EPC + e];
+                        }
+#pragma unroll
+                        for (int e = 0; e < EPC; ++e) d[u] = fmaf(qs[c * EPC + e], f[e], d[u]);
+                    }
+                }
+#pragma unroll
+                for (int u = 0; u < 4; ++u) {
+                    for (int o = lk >> 1; o > 0; o >>= 1) d[u] += __shfl_xor_sync(0xffffffffu, d[u], o);
+                    const int j = j0 + u * side + lane / lk;
+                    if (kch == 0 && j < 8) ps[8 * warp + j] = d[u];
+                }
+            }
+            __syncthreads();
+            // every warp takes the tile's 32 scores, one per lane
+            const int t = tb + lane;
+            const float sc = t < t1 ? ps[lane] - slope * (float)(pos - t) : NEG;
+            const float mn = fmaxf(m, warp_max(sc));
+            const float pr = t < t1 ? expf(sc - mn) : 0.0f, corr = expf(m - mn);
+            l = l * corr + warp_sum(pr);
+            m = mn;
+            __syncthreads();
+            if (warp == 0) ps[lane] = pr;
+            __syncthreads();
+#pragma unroll
+            for (int e = 0; e < 8; ++e) acc[e] *= corr;
+            if (vch < nvc) {
+                const int nt = min(MIX_TILE, t1 - tb);
+#pragma unroll 4
+                for (int j = vgrp; j < nt; j += vgroups) {
+                    const int tt = tb + j;
+                    float f[EPC];
+                    if (tt == pos) {
+#pragma unroll
+                        for (int e = 0; e < EPC; ++e) f[e] = vc[vch * EPC + e];
+                    } else {
+                        const int page = p.page_table[tt / a.page_tokens];
+                        Elem<KT>::unpack(ldg_stream_coherent(pool + a.v_at(page, g, tt % a.page_tokens) + (size_t)vch * EPC), f);
+                    }
+                    const float w = ps[j];
+#pragma unroll
+                    for (int e = 0; e < EPC; ++e) acc[e] = fmaf(w, f[e], acc[e]);
+                }
+            }
+            __syncthreads();
+        }
+#pragma unroll
+        for (int e = 0; e < 8; ++e) accs[tid * 8 + e] = acc[e];
+        __syncthreads();
+        float* pa = p.part_acc + ((size_t)h * p.nsplit + sl) * a.vp;
+        for (int i = tid; i < a.vp; i += MIX_THREADS) {
+            float s = 0.0f;
+            for (int gg = 0; gg < vgroups; ++gg) s += accs[(gg * lv + i / EPC) * 8 + i % EPC];
+            pa[i] = s;
+        }
+    }
+    if (tid == 0) {
+        p.part_ml[((size_t)h * p.nsplit + sl) * 2] = m;
+        p.part_ml[((size_t)h * p.nsplit + sl) * 2 + 1] = l;
+    }
+    __threadfence();
+    __syncthreads();
+    if (tid == 0) s_last = atomicAdd(&p.counters[h], 1u) == (unsigned)p.nsplit - 1u;
+    __syncthreads();
+    if (!s_last) return;
+    __threadfence();
+    const float sink = p.sink[h];
+    float ms = NEG, ls = 0.0f;  // nsplit <= 32: one slice per lane, the same in every warp
+    if (lane < p.nsplit) {
+        const float2 ml = __ldcg(reinterpret_cast<const float2*>(p.part_ml + ((size_t)h * p.nsplit + lane) * 2));
+        ms = ml.x;
+        ls = ml.y;
+    }
+    const float M = fmaxf(warp_max(ls > 0.0f ? ms : NEG), sink);
+    const float w = ls > 0.0f ? expf(ms - M) : 0.0f;
+    const float L = warp_sum(ls * w) + expf(sink - M);
+    const float inv = sigmoid(__ldcg(p.proj + p.pl.lg + h)) / L;
+    if (warp == 0) ps[lane] = w;
+    __syncthreads();
+    const int used = (len + per - 1) / per;  // slices that hold positions
+    for (int i = tid; i < a.vdim; i += MIX_THREADS) {
+        float o = 0.0f;
+#pragma unroll 4
+        for (int s = 0; s < used; ++s) o = fmaf(__ldcg(p.part_acc + ((size_t)h * p.nsplit + s) * a.vp + i), ps[s], o);
+        p.attn[h * a.vdim + i] = o * inv;
+    }
+    if (tid == 0) p.counters[h] = 0u;
+}
+
+// grid = Hr * nslice memory CTAs, then H * nsplit attention CTAs
+template <typename KT>
+__global__ void __launch_bounds__(MIX_THREADS) mixer_step_kernel(const __grid_constant__ MixerStep p, KT* __restrict__ pool) {
+    extern __shared__ float mix_sm[];
+    __shared__ float red[32];
+    __shared__ int s_last;
+    const int nmem = p.d.H * p.d.nslice;
+    if ((int)blockIdx.x < nmem) mem_step(p, blockIdx.x, mix_sm, red);
+    else attn_step<KT>(p, pool, blockIdx.x - nmem, mix_sm, red, s_last);
+}
+
+}  // namespace cd

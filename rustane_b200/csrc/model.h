@@ -19,8 +19,36 @@ struct cd_layer_dev {
     void* kv;     // this layer's pages: [num_pages][2][kv_heads][page_tokens][hd]
 };
 
+struct cd_model;
+
 enum cd_head_mode { HEAD_NONE = 0, HEAD_LOGITS, HEAD_ARGMAX, HEAD_TOPK, HEAD_STATS,
                     LOOP_GREEDY, LOOP_TOPK, LOOP_FULLVOCAB };
+
+// one step of the token loop
+struct cd_step {
+    int input;  // 0: x already in x_a; 1: embed st->token; 2: take the next prompt token, then embed
+    int head;   // cd_head_mode
+    int k = 0;
+    float t = 0.f, softcap = 0.f, inv_t = 1.f;
+};
+
+// A model family: how its layers are stepped and what it keeps per sequence besides the shared cache.  The token loop,
+// the samplers, the session and the C ABI (model.cu, session.cpp) drive every family through this table; a null
+// entry means the family has no such path (the callers then take the one-token-at-a-time one, or report it).
+struct cd_family {
+    const char* name;
+    cudaError_t (*enqueue_step)(cd_model*, const cd_step&);
+    cudaError_t (*enqueue_head_only)(cd_model*);         // final norm + LM head on x_a
+    int (*prefill)(cd_model*, size_t n);                 // the prompt tokens in prompt_dev together; x_a = the last one's hidden state
+    const float* (*hidden_row)(const cd_model*, size_t); // hidden state of token i of the last such pass
+    int (*samples)(cd_model*, const uint32_t* first, int ns, size_t nsteps, int mode, int top_k, float t, float softcap, uint64_t* rng, uint32_t* out_ids);
+    void (*release)(cd_model*);
+    // recurrent state (rewinding cannot just forget cached rows): `mark` keeps the state at the current length, `can_rewind`
+    // tells whether the state at `len` is still known, `rewind` goes back to it
+    int (*mark)(cd_model*);
+    bool (*can_rewind)(const cd_model*, size_t len);
+    int (*rewind)(cd_model*, size_t len);
+};
 
 struct cd_graph_key {
     int mode, k, input;
@@ -76,7 +104,14 @@ struct cd_moe_state {
     bool stream_ffn = false;        // the experts' rows go through the streamed GEMV (else: the plain-load kernels)
 };
 
+struct cd_hybrid_state;  // hybrid.h: a decoder whose layers a configuration file lists
+
 struct cd_model {
+    const cd_family* family = nullptr;
+    cd_hybrid_state* hybrid = nullptr;  // set: the handle is a configured decoder (hybrid.h)
+    bool replicated_head = false;       // several ranks, each with the whole LM head (expert parallelism)
+    float rms_eps = cd::RMS_EPS;        // of the norm ahead of the LM head
+    size_t state_len = 0;               // tokens the recurrent state has seen (families that keep one); SIZE_MAX: unknown
     cd_moe_state* moe = nullptr;  // set: the handle is a MoE + MLA decoder
     cd_config cfg;       // what this GPU holds: under tensor parallelism heads, kv_heads, hidden, q_dim, kv_dim are per rank
     cd_config full_cfg;  // the model as the caller described it
@@ -117,17 +152,18 @@ struct cd_model {
     size_t len = 0;
 
     // weights
-    void* weight_arena = nullptr;
+    void* weight_arena = nullptr;  // embedding, LM head, final gamma
+    void* layer_arena = nullptr;   // the layers' matrices
     size_t weight_bytes = 0;
     void* embed = nullptr;
     void* lm_head = nullptr;  // == embed when tied
     float* gamma_final = nullptr;
     std::vector<cd_layer_dev> layers;
     void* kv_arena = nullptr;
-    size_t kv_layer_bytes = 0;
 
     // workspace
     void* ws_arena = nullptr;
+    char* family_ws = nullptr;  // AllocSpec::family_ws_bytes of it
     float *x_a = nullptr, *x_b = nullptr, *q = nullptr, *attn = nullptr, *gate = nullptr;
     float *logits = nullptr, *logits_capped = nullptr, *norm_final = nullptr, *part_acc = nullptr, *part_ml = nullptr;
     unsigned int* counters = nullptr;  // [heads] attention + [1] head
@@ -165,9 +201,21 @@ namespace cd {
 int fail(cd_model* m, int code, const std::string& msg);
 int device_wait_failed(cd_model* m, int dev_code, const char* where);
 void set_global_error(const std::string& msg);
-// builder: allocate, fill tensors given in the reference's layouts, finish
-int model_alloc(const cd_config* cfg, const cd_options* opts, int untied, cd_model** out, const cd_moe_config* moe = nullptr);
-void moe_release(cd_model* m);
+// What a family asks of the shared allocation: embedding, LM head, cache pages, workspace, head scratch, device state.
+struct AllocSpec {
+    const cd_family* family = nullptr;
+    cd_config local;                    // what this GPU holds (== cfg on one GPU)
+    bool sharded_head = false;          // the LM head is split by vocabulary blocks over the ranks
+    std::vector<size_t> kv_row_elems;   // per layer: cached elements per position
+    int rope_dim = 0;                   // width the RoPE pairs run over; 0: no table
+    int attn_parts = 1;                 // attention partials per head the family's kernels may leave (at least)
+    size_t family_ws_bytes = 0;         // device scratch of the family's own (cd_model::family_ws), zero-filled
+    size_t tp_prefill_rows = 0;         // prompt rows of the tensor-parallel partial-sum buffers
+};
+int resolve_kv_dtype(const cd_options& opts, int* kv_dtype);
+int model_alloc(const cd_config* cfg, const cd_options& opts, int untied, const AllocSpec& spec, cd_model** out);
+// dense family (dense.cu): allocate, fill tensors given in the reference's layouts
+int dense_alloc(const cd_config* cfg, const cd_options* opts, int untied, cd_model** out);
 size_t model_tensor_elems(const cd_model* m, int which);
 int model_set_tensor_f32(cd_model* m, int layer, int which, const float* host);
 int model_set_tensor_synth(cd_model* m, int layer, int which, uint64_t seed, float std);
@@ -177,9 +225,13 @@ int model_set_quant_rows(cd_model* m, int layer, int which, const void* host);
 int model_get_quant_rows(cd_model* m, int layer, int which, void* host, size_t cap);
 int model_get_plain(cd_model* m, int layer, int which, void* host, size_t cap);
 int model_finish(cd_model* m);
-// batched prompt pass (prefill.cu): on CD_OK the cache holds positions len .. len+n-1 of the prompt in
+int check_room(cd_model* m, size_t need);
+int set_state(cd_model* m, uint32_t token);
+void count_launch(cd_model* m);
+// the dense family's batched prompt pass (prefill.cu): on CD_OK the cache holds positions len .. len+n-1 of the prompt in
 // m->prompt_dev and m->x_a holds the last position's hidden state; CD_ERR_UNSUPPORTED: use the per-token path
 int prefill_batched(cd_model* m, size_t n);
+const float* prefill_hidden_row(const cd_model* m, size_t i);
 void prefill_release(cd_model* m);
 // ns samples continuing the cached prompt together (prefill.cu); mode 0 greedy, 1 top-k, 2 full-vocabulary
 int decode_samples(cd_model* m, const uint32_t* first, int ns, size_t nsteps, int mode, int top_k, float t, float softcap, uint64_t* rng,

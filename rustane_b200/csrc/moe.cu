@@ -1,20 +1,17 @@
 // Construction of the MoE + MLA decoder (cd_moe_model_create_synthetic): device memory for its
-// weights and scratch, synthetic tensors generated in place.  The step itself is enqueued by
-// model.cu (enqueue_step_moe_t) from the kernels of moe.cuh.  No reference counterpart.
+// weights and scratch, synthetic tensors generated in place, and its per-token step (enqueue_step_moe_t)
+// from the kernels of moe.cuh.  No reference counterpart.
 #include <algorithm>
+#include <cmath>
 #include <cstring>
 #include <vector>
 
-#include "kernels.cuh"
+#include "step.cuh"
 #include "moe.cuh"
-#include "model.h"
 
 using namespace cd;
 
 namespace {
-
-inline size_t align_up(size_t v, size_t a) { return (v + a - 1) / a * a; }
-inline size_t esize(int dtype) { return dtype == CD_DTYPE_F32 ? 4 : 2; }
 
 // tensor ids of the synthetic generator: uid = 0x100000 + 1024 * layer + local
 enum { L_WQ = 0, L_WDKV, L_WKR, L_WUK, L_WUV, L_WO, L_WR, L_WS1, L_WS3, L_WS2, L_EXPERT0 = 16 };
@@ -78,9 +75,6 @@ int build(cd_model* m, uint64_t seed, float std, int untied) {
     return CD_OK;
 }
 
-}  // namespace
-
-namespace cd {
 void moe_release(cd_model* m) {
     if (!m->moe) return;
     if (m->moe->arena) cudaFree(m->moe->arena);
@@ -88,15 +82,150 @@ void moe_release(cd_model* m) {
     delete m->moe;
     m->moe = nullptr;
 }
-}  // namespace cd
+
+// One token through the MoE + MLA decoder (moe.cuh).  WT: storage of all weights; KT: storage of the latent cache.
+template <typename WT, typename KT>
+cudaError_t enqueue_step_moe_t(cd_model* m, const cd_step& p) {
+    const cd_config& c = m->cfg;
+    cd_moe_state& S = *m->moe;
+    const cd_moe_config& mc = S.mc;
+    cudaError_t e;
+#define TRY(x) do { e = (x); if (e != cudaSuccess) return e; } while (0)
+    m->cur_cls = CLS_MISC;
+    m->next_stream.w = nullptr;
+    if (p.input == 2) {
+        next_prompt_kernel<<<1, 1, 0, m->stream>>>(m->st, m->prompt_dev);
+        count_launch(m);
+    }
+    if (p.input >= 1) {
+        embed_kernel<WT><<<std::max(1, c.dim / 256), 256, 0, m->stream>>>((const WT*)m->embed, m->st, m->x_a, c.dim, m->full_cfg.vocab);
+        count_launch(m);
+        TRY(cudaGetLastError());
+    }
+    const MlaDims md{c.heads, mc.kv_latent, mc.rope_dim, mc.nope_dim, mc.v_dim, m->page_tokens};
+    const MoeDims ed{c.dim, c.hidden, S.shared_cols};
+    const MoePick pick{S.loc_ids, S.loc_w, S.n_loc};
+    const int W = mc.kv_latent + mc.rope_dim, QA = c.q_dim + W, units = mc.top_k * c.hidden + S.shared_cols;
+    const bool ep = m->tp_world > 1;
+    const float scale = 1.0f / std::sqrt((float)c.hd);
+    // the tensor-core attention takes a 16-bit cache of the 512-wide latent geometry; anything else the plain kernel
+    const bool attn_mma = !std::is_same<KT, float>::value && mc.kv_latent == MLA_MMA_C && W % 16 == 0 && c.heads <= 16;
+    const size_t attn_smem = attn_mma ? mla_mma_smem_bytes(W)
+                                      : ((size_t)(c.heads + MLA_TILE) * (W + 1) + (size_t)c.heads * MLA_TILE + 3 * c.heads) * sizeof(float);
+    static size_t attn_set = 0, w2_set = 0;  // per instantiation
+    if (attn_smem > attn_set) {
+        if constexpr (!std::is_same<KT, float>::value) TRY(cudaFuncSetAttribute(mla_attn_mma_kernel<KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)std::max(attn_smem, mla_mma_smem_bytes(W))));
+        TRY(cudaFuncSetAttribute(mla_attn_kernel<KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)attn_smem));
+        attn_set = attn_smem;
+    }
+    if (!S.stream_ffn && (size_t)units * 4 > w2_set) {
+        TRY(cudaFuncSetAttribute(moe_w2_kernel<WT>, cudaFuncAttributeMaxDynamicSharedMemorySize, units * 4));
+        w2_set = (size_t)units * 4;
+    }
+    const uint32_t es = (uint32_t)sizeof(WT);
+    for (int l = 0; l < c.nlayers; ++l) {
+        const cd_moe_layer_dev& L = S.layers[l];
+        int* sel = S.sel_ids + (size_t)l * mc.top_k;
+        m->cur_cls = CLS_QKV;
+        if (ep && l > 0) { m->tp_in.in_reduce = l; m->tp_in.res = m->x_b; m->tp_in.x_out = m->x_a; }  // x = x2 + alpha * sum(ranks' FFN partials)
+        TRY((launch_gemv<WT, 1, true>(m, L.wqa, m->x_a, L.gamma1, nullptr, QA, c.dim, EpiStore{S.qa})));
+        m->cur_cls = CLS_ATTN;
+        TRY(launch_chain(m, mla_post_kernel<WT, KT>, dim3((c.heads * mc.kv_latent + 127) / 128 + 1), dim3(128), std::max(c.heads * mc.nope_dim, mc.kv_latent) * sizeof(float),
+                         (const float*)S.qa, (const WT*)L.wuk_t, (const float*)L.gamma_kv, (const float2*)m->rope, (const int*)m->page_table, (const DevState*)m->st,
+                         (KT*)m->layers[l].kv, S.qabs, attn_mma ? (KT*)S.qsplit : (KT*)nullptr, md));
+        if constexpr (!std::is_same<KT, float>::value) {
+            if (attn_mma)
+                TRY(launch_chain(m, mla_attn_mma_kernel<KT>, dim3(S.nsplit), dim3(MLA_MMA_THREADS), attn_smem, (const KT*)S.qsplit, (const KT*)m->layers[l].kv,
+                                 (const int*)m->page_table, (const DevState*)m->st, S.part_acc, S.part_ml, md, S.nsplit, scale, &m->st->error));
+        }
+        if (!attn_mma)
+            TRY(launch_chain(m, mla_attn_kernel<KT>, dim3(S.nsplit), dim3(256), attn_smem, (const float*)S.qabs, (const KT*)m->layers[l].kv, (const int*)m->page_table,
+                             (const DevState*)m->st, S.part_acc, S.part_ml, md, S.nsplit, scale));
+        TRY(launch_chain(m, mla_out_kernel<WT>, dim3(c.heads, (mc.v_dim + 31) / 32), dim3(256), (mc.kv_latent + S.nsplit) * sizeof(float), (const float*)S.part_acc,
+                         (const float*)S.part_ml, (const WT*)L.wuv_t, m->attn, (const DevState*)m->st, md, S.nsplit, attn_mma ? MLA_MMA_TILE : MLA_TILE));
+        m->cur_cls = CLS_WO;
+        TRY((launch_gemv<WT, 1, false>(m, L.wo, m->attn, nullptr, nullptr, c.dim, c.heads * mc.v_dim, EpiResidual{m->x_a, m->x_b, m->alpha})));
+        m->cur_cls = CLS_W13;
+        TRY(launch_chain(m, moe_router_kernel<WT, RouterRmsIn>, dim3((mc.n_experts + 3) / 4), dim3(128), std::max(c.dim, mc.n_experts + 1) * sizeof(float),
+                         RouterRmsIn{m->x_b, L.gamma2, S.xn2}, (const WT*)L.wr, S.router_logits, S.router_counter, sel, S.sel_w, S.loc_ids, S.loc_w, S.n_loc, c.dim,
+                         RouteRule{mc.n_experts, mc.top_k, 1, 1}, S.e0, S.n_local));
+        TpLink tp = m->tp;
+        tp.ar_out = l + 1;
+        if (S.stream_ffn) {
+            // the chosen experts' rows gathered by the streamed GEMV's copy engine; K and N are upper bounds (all top_k local)
+            const SrcExpertRows s13{S.loc_ids, S.n_loc, L.ws13, 2 * c.hidden, 2 * S.shared_cols};
+            TRY((launch_gemv<WT, 2, false>(m, L.w13, S.xn2, nullptr, nullptr, 2 * units, c.dim, EpiGateMoe{S.gate, S.loc_w, S.n_loc, c.hidden}, s13)));
+            m->cur_cls = CLS_W2;
+            const SrcExpertCols s2{S.loc_ids, S.n_loc, L.ws2, c.hidden, S.shared_cols, c.dim, (uint32_t)c.hidden * es, (uint32_t)S.shared_cols * es};
+            if (ep) TRY((launch_gemv<WT, 1, false>(m, L.w2, S.gate, nullptr, nullptr, c.dim, units, EpiPush{tp}, s2)));
+            else TRY((launch_gemv<WT, 1, false>(m, L.w2, S.gate, nullptr, nullptr, c.dim, units, EpiResidual{m->x_b, m->x_a, m->alpha}, s2)));
+        } else {
+            TRY(launch_chain(m, moe_w13_kernel<WT>, dim3((units + 7) / 8), dim3(256), c.dim * sizeof(float), (const float*)S.xn2, (const WT*)L.w13, (const WT*)L.ws13, pick,
+                             S.gate, ed));
+            m->cur_cls = CLS_W2;
+            TRY(launch_chain(m, moe_w2_kernel<WT>, dim3((c.dim + 7) / 8), dim3(256), units * sizeof(float), (const float*)S.gate, (const WT*)L.w2, (const WT*)L.ws2, pick,
+                             (const float*)m->x_b, m->x_a, m->alpha, ed, ep ? tp : TpLink{}));
+        }
+        TRY(cudaGetLastError());
+    }
+    return enqueue_head_t<WT, WT>(m, p, false, ep ? (unsigned int)c.nlayers : 0u, c.nlayers);
+#undef TRY
+}
+
+cudaError_t moe_step(cd_model* m, const cd_step& p) {
+    switch (m->opt.weight_dtype) {
+        case CD_DTYPE_F32: return enqueue_step_moe_t<float, float>(m, p);
+        case CD_DTYPE_F16: return enqueue_step_moe_t<__half, __half>(m, p);
+        default: return m->kv_dtype == CD_DTYPE_F16 ? enqueue_step_moe_t<__nv_bfloat16, __half>(m, p) : enqueue_step_moe_t<__nv_bfloat16, __nv_bfloat16>(m, p);
+    }
+}
+
+cudaError_t moe_head_only(cd_model* m) {
+    cudaError_t e = cudaSuccess;
+    DISPATCH_WT(m->opt.weight_dtype, WT, e = enqueue_head_only_t<WT>(m));
+    return e;
+}
+
+const cd_family MOE_FAMILY = {"moe_mla", moe_step, moe_head_only, nullptr, nullptr, nullptr, moe_release, nullptr, nullptr, nullptr};
+
+int validate_moe(const cd_config& c, const cd_moe_config& mc, int dtype, int world) {
+    if (c.dim <= 0 || c.hidden <= 0 || c.heads <= 0 || c.seq <= 0 || c.nlayers <= 0 || c.vocab <= 0 || mc.n_experts <= 0 || mc.top_k <= 0 ||
+        mc.n_shared < 0 || mc.kv_latent <= 0 || mc.rope_dim <= 0 || mc.nope_dim <= 0 || mc.v_dim <= 0)
+        return fail(nullptr, CD_ERR_INVALID, "config contains a non-positive dimension");
+    if (c.hd != mc.nope_dim + mc.rope_dim || c.q_dim != c.heads * c.hd || c.kv_dim != mc.kv_latent + mc.rope_dim || c.kv_heads != 1 || c.gqa_ratio != c.heads)
+        return fail(nullptr, CD_ERR_INVALID, "cd_config of a MoE + MLA model: hd = nope_dim + rope_dim, q_dim = heads * hd, kv_dim = kv_latent + rope_dim, kv_heads = 1, gqa_ratio = heads");
+    if (dtype != CD_DTYPE_F32 && dtype != CD_DTYPE_F16 && dtype != CD_DTYPE_BF16) return fail(nullptr, CD_ERR_UNSUPPORTED, "MoE + MLA weights are f32, f16 or bf16");
+    if (mc.top_k > mc.n_experts || mc.top_k > 16) return fail(nullptr, CD_ERR_INVALID, "top_k must not exceed n_experts (and 16)");
+    if (c.heads > MLA_MAX_HEADS || mc.kv_latent > 512) return fail(nullptr, CD_ERR_UNSUPPORTED, "MLA attention supports at most 16 heads and a latent of 512");
+    const int epc = dtype == CD_DTYPE_F32 ? 4 : 8;
+    if (c.dim % 8 || c.hidden % 8 || mc.kv_latent % 8 || mc.rope_dim % 8 || mc.nope_dim % 8 || mc.v_dim % 8 || (c.heads * mc.v_dim) % 8)
+        return fail(nullptr, CD_ERR_UNSUPPORTED, "dim, hidden and the MLA widths must be multiples of 8");
+    if (c.dim > 8 * 256 * epc || c.heads * mc.v_dim > 8 * 256 * epc) return fail(nullptr, CD_ERR_UNSUPPORTED, "inner dimension too large for the GEMV tiling");
+    if (world > 1 && (mc.n_experts % world || (mc.n_shared * c.hidden) % (8 * world)))
+        return fail(nullptr, CD_ERR_UNSUPPORTED, "n_experts and the shared FFN's columns / 8 must be divisible by the expert-parallel world size");
+    return CD_OK;
+}
+}  // namespace
 
 extern "C" int cd_moe_model_create_synthetic(const cd_config* cfg, const cd_moe_config* moe, const cd_options* opts, uint64_t seed, float std,
                                              int untied_head, cd_model** out) {
     if (!cfg || !moe || !out) return fail(nullptr, CD_ERR_INVALID, "null argument");
     *out = nullptr;
-    cd_model* m = nullptr;
-    int rc = model_alloc(cfg, opts, untied_head != 0, &m, moe);
+    cd_options o;
+    memset(&o, 0, sizeof(o));
+    o.device = -1;
+    if (opts) o = *opts;
+    const int world = std::max(1, (int)o.tp_world);
+    int rc = validate_moe(*cfg, *moe, o.weight_dtype, world);
     if (rc) return rc;
+    if (world > 1 && (world > TP_MAX || o.tp_rank < 0 || o.tp_rank >= world)) return fail(nullptr, CD_ERR_INVALID, "expert-parallel rank / world out of range");
+    AllocSpec spec;
+    spec.family = &MOE_FAMILY;
+    spec.local = *cfg;
+    spec.kv_row_elems.assign(cfg->nlayers, (size_t)cfg->kv_dim);  // one [latent | rope key] row per position
+    spec.rope_dim = moe->rope_dim;
+    cd_model* m = nullptr;
+    if ((rc = model_alloc(cfg, o, untied_head != 0, spec, &m))) return rc;
     auto bail = [&](int code) { set_global_error(m->err); cd_model_destroy(m); return code; };
     const cd_config& c = m->cfg;
     cd_moe_state* S = new cd_moe_state();

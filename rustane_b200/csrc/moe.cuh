@@ -545,23 +545,133 @@ mla_attn_mma_kernel(const KT* __restrict__ qsplit, const KT* __restrict__ lat_po
     }
 }
 
+// ---------------------------------------------------------------------- routing rule
+struct RouteRule {
+    int experts, top;
+    int groups, keep;  // experts form `groups` equal runs of neighbours; only the `keep` runs whose best score is largest may be chosen from
+};
+// One warp picks a token's experts: pr[experts] holds the router logits (shared memory, rewritten), gs[groups] is scratch.
+// Scores are softmax(logits) over all experts; ties go to the lower index; each(k, expert, score)
+// is called in every lane with the k-th choice and its score, unchanged.
+template <class Each>
+__device__ inline void route_pick(float* pr, float* gs, const RouteRule& r, int lane, Each each) {
+    float mx = -INFINITY;
+    for (int k = lane; k < r.experts; k += 32) mx = fmaxf(mx, pr[k]);
+    mx = warp_max(mx);
+    __syncwarp();
+    for (int k = lane; k < r.experts; k += 32) pr[k] = expf(pr[k] - mx);
+    __syncwarp();
+    float sum = 0.0f;  // in expert order, the same in every lane
+    for (int k = 0; k < r.experts; ++k) sum += pr[k];
+    __syncwarp();
+    for (int k = lane; k < r.experts; k += 32) pr[k] = pr[k] / sum;
+    __syncwarp();
+    auto best = [&](const float* v, int n, float& bv, int& bi) {
+        bv = -INFINITY;
+        bi = 0x7fffffff;
+        for (int i = lane; i < n; i += 32) {
+            const float t = v[i];
+            if (t > bv || (t == bv && i < bi)) { bv = t; bi = i; }
+        }
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
+            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+            if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
+        }
+        if (bi >= n) bi = 0;  // nothing comparable (NaN logits): never an address past the list
+    };
+    float bv;
+    int bi;
+    if (r.keep < r.groups) {
+        const int size = r.experts / r.groups;
+        for (int g = lane; g < r.groups; g += 32) {
+            float t = -INFINITY;
+            for (int i = 0; i < size; ++i) t = fmaxf(t, pr[g * size + i]);
+            gs[g] = t;
+        }
+        __syncwarp();
+        for (int k = 0; k < r.keep; ++k) {
+            best(gs, r.groups, bv, bi);
+            __syncwarp();
+            if (lane == 0) gs[bi] = -INFINITY;  // kept
+            __syncwarp();
+        }
+        for (int i = lane; i < r.experts; i += 32)
+            if (gs[i / size] != -INFINITY) pr[i] = -1.0f;  // scores are never negative: below any expert that may be chosen
+        __syncwarp();
+    }
+    for (int k = 0; k < r.top; ++k) {
+        best(pr, r.experts, bv, bi);
+        each(k, bi, bv);
+        __syncwarp();
+        if (lane == 0) pr[bi] = -INFINITY;  // removed from the later rounds
+        __syncwarp();
+    }
+}
+
+// What the router multiplies: fill(xs) writes the vector to shared memory (all threads; the barriers of the block
+// reductions publish it) and returns the factor its dot products still need; CTA 0 keeps the vector for the expert kernels.
+struct RouterRmsIn {  // rmsnorm(x, gamma)
+    const float *x, *gamma;
+    float* out;
+    __device__ float fill(float* xs, float* red, int dim, bool writer) const {
+        float ss = 0.0f;
+        for (int i = threadIdx.x; i < dim; i += blockDim.x) {
+            const float v = __ldcg(x + i);
+            xs[i] = v * gamma[i];
+            ss += v * v;
+        }
+        const float inv = 1.0f / sqrtf(block_sum(ss, red) * (1.0f / (float)dim) + RMS_EPS);
+        if (writer)
+            for (int i = threadIdx.x; i < dim; i += blockDim.x) out[i] = xs[i] * inv;
+        return inv;
+    }
+};
+struct RouterMixIn {  // the residual stream behind two parallel mixers (InParallelMix, mixers.cuh)
+    const float *x, *yl, *yr, *wl, *wr, *gain;
+    float* out;
+    float mult, eps;
+    __device__ float fill(float* xs, float* red, int dim, bool writer) const {
+        float sl = 0.0f, sr = 0.0f, ss = 0.0f;
+        for (int i = threadIdx.x; i < dim; i += blockDim.x) {
+            const float a = __ldcg(yl + i), b = __ldcg(yr + i);
+            sl = fmaf(a, a, sl);
+            sr = fmaf(b, b, sr);
+        }
+        const float rl = 0.5f / sqrtf(block_sum(sl, red) * (1.0f / (float)dim) + eps);
+        const float rr = 0.5f / sqrtf(block_sum(sr, red) * (1.0f / (float)dim) + eps);
+        for (int i = threadIdx.x; i < dim; i += blockDim.x) {
+            const float z = __ldcg(yl + i) * rl * wl[i] + __ldcg(yr + i) * rr * wr[i];
+            xs[i] = z;
+            ss = fmaf(z, z, ss);
+        }
+        const float r = mult / sqrtf(block_sum(ss, red) * (1.0f / (float)dim) + eps);
+        for (int i = threadIdx.x; i < dim; i += blockDim.x) {
+            const float v = __ldcg(x + i) + xs[i] * r * gain[i];
+            xs[i] = v;
+            if (writer) out[i] = v;
+        }
+        __syncthreads();
+        return 1.0f;
+    }
+};
+
 // ---------------------------------------------------------------------- router: one warp per expert, the last CTA picks
-// xn = rmsnorm(x, gamma) (every CTA, CTA 0 keeps it for the expert kernels), logit_e = W_r[e] . xn;
-// the CTA that finishes last (a counter, nobody waits) computes p = softmax(logits) and the top_k
-// largest p (k rounds of arg-max, ties to the lower expert index) with their weights, not
-// renormalised.  Besides the choice (sel_ids, sel_w) it writes the compact list of the chosen experts
+// logit_e = W_r[e] . xn (every CTA forms xn, see above); the CTA that finishes last (a counter, nobody waits) applies the
+// routing rule.  Besides the choice (sel_ids, sel_w) it writes the compact list of the chosen experts
 // this rank holds (local index, weight, count): the expert kernels walk that list.
-template <typename WT>
+template <typename WT, class In>
 __global__ void __launch_bounds__(128)
-moe_router_kernel(const float* __restrict__ x, const float* __restrict__ gamma, const WT* __restrict__ wr, float* __restrict__ xn_out,
-                  float* __restrict__ logits, unsigned int* __restrict__ counter, int* __restrict__ sel_ids, float* __restrict__ sel_w,
-                  int* __restrict__ loc_ids, float* __restrict__ loc_w, int* __restrict__ n_loc, int dim, int n_experts, int top_k, int e0,
-                  int n_local) {
-    extern __shared__ float sm[];  // [dim] x * gamma; the last CTA: [n_experts] probabilities on top of it
+moe_router_kernel(In in, const WT* __restrict__ wr, float* __restrict__ logits, unsigned int* __restrict__ counter, int* __restrict__ sel_ids,
+                  float* __restrict__ sel_w, int* __restrict__ loc_ids, float* __restrict__ loc_w, int* __restrict__ n_loc, int dim, RouteRule rule,
+                  int e0, int n_local) {
+    extern __shared__ float sm[];  // [dim] the input; the last CTA: [experts] scores and [groups] on top of it
     __shared__ float red[32];
     __shared__ int s_last;
     constexpr int EPC = Elem<WT>::EPC, PRE = 8;
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nw = blockDim.x >> 5;
+    const int n_experts = rule.experts;
     float* xg = sm;
     // this warp's expert row: its first chunks are requested before anything else (x, gamma and the row arrive together)
     const int e = min(blockIdx.x * nw + warp, n_experts - 1);
@@ -572,17 +682,7 @@ moe_router_kernel(const float* __restrict__ x, const float* __restrict__ gamma, 
     for (int j = 0; j < PRE; ++j) w[j] = lane + 32 * j < nchunks ? ldg_stream(row + (size_t)(lane + 32 * j) * 16) : make_uint4(0, 0, 0, 0);
     pdl_wait();
     pdl_launch_dependents();  // after the wait: at most this kernel and the next one overlap
-    float ss = 0.0f;
-    for (int i = tid; i < dim; i += blockDim.x) {
-        const float v = __ldcg(x + i);
-        xg[i] = v * gamma[i];
-        ss += v * v;
-    }
-    const float tot = block_sum(ss, red);  // (its barriers also publish xg)
-    const float inv = 1.0f / sqrtf(tot * (1.0f / (float)dim) + RMS_EPS);
-    if (blockIdx.x == 0)
-        for (int i = tid; i < dim; i += blockDim.x) xn_out[i] = xg[i] * inv;
-    // logit = inv * (row . (x * gamma))
+    const float inv = in.fill(xg, red, dim, blockIdx.x == 0);
     float a = 0.0f;
 #pragma unroll
     for (int j = 0; j < PRE; ++j) {
@@ -608,45 +708,19 @@ moe_router_kernel(const float* __restrict__ x, const float* __restrict__ gamma, 
     __syncthreads();
     if (!s_last || warp != 0) return;
     __threadfence();
-    float* pr = sm;  // x * gamma is no longer needed: the other warps have left, this one has its logit
-    float mx = -INFINITY;
-    for (int k = lane; k < n_experts; k += 32) {
-        const float v = __ldcg(logits + k);
-        pr[k] = v;
-        mx = fmaxf(mx, v);
-    }
-    mx = warp_max(mx);
-    __syncwarp();
-    for (int k = lane; k < n_experts; k += 32) pr[k] = expf(pr[k] - mx);
-    __syncwarp();
-    float sum = 0.0f;  // in expert order, the same in every lane
-    for (int k = 0; k < n_experts; ++k) sum += pr[k];
-    __syncwarp();
-    for (int k = lane; k < n_experts; k += 32) pr[k] = pr[k] / sum;
+    float* pr = sm;  // the input is no longer needed: the other warps have left, this one has its logit
+    for (int k = lane; k < n_experts; k += 32) pr[k] = __ldcg(logits + k);
     __syncwarp();
     int nl = 0;
-    for (int k = 0; k < top_k; ++k) {
-        float bv = -INFINITY;
-        int bi = 0x7fffffff;
-        for (int i = lane; i < n_experts; i += 32) {
-            const float v = pr[i];
-            if (v > bv || (v == bv && i < bi)) { bv = v; bi = i; }
-        }
-#pragma unroll
-        for (int o = 16; o > 0; o >>= 1) {
-            const float ov = __shfl_xor_sync(0xffffffffu, bv, o);
-            const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-            if (ov > bv || (ov == bv && oi < bi)) { bv = ov; bi = oi; }
-        }
+    route_pick(pr, pr + n_experts, rule, lane, [&](int k, int bi, float bv) {
+        const bool here = bi >= e0 && bi < e0 + n_local;
         if (lane == 0) {
             sel_ids[k] = bi;
             sel_w[k] = bv;
-            pr[bi] = -INFINITY;  // removed from the later rounds
-            if (bi >= e0 && bi < e0 + n_local) { loc_ids[nl] = bi - e0; loc_w[nl] = bv; }
+            if (here) { loc_ids[nl] = bi - e0; loc_w[nl] = bv; }
         }
-        if (bi >= e0 && bi < e0 + n_local) ++nl;  // bi is the same in every lane after the exchange
-        __syncwarp();
-    }
+        if (here) ++nl;  // bi is the same in every lane
+    });
     if (lane == 0) {
         *n_loc = nl;
         *counter = 0u;  // for the next launch

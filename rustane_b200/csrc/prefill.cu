@@ -4,7 +4,7 @@
 // residual stream in fp32 and 16-bit GEMM inputs; K and V go straight into the pages the
 // decode kernels read.  Used by cd_prefill for bf16 / fp16 models on one GPU; every other
 // case keeps feeding the prompt one token at a time.
-#include "prefill.cuh"
+#include "pf_launch.cuh"
 
 #include <algorithm>
 #include <cmath>
@@ -18,10 +18,6 @@
 
 namespace cd {
 namespace {
-
-typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*,
-                                  const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
-                                  CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
 struct SampleGraphKey {
     int ns = 0, mode = 0, top_k = 0;
@@ -65,18 +61,6 @@ struct PrefillCtx {
     void* vt = nullptr;       // [kv_heads * hd][key_ld]
 };
 
-inline size_t round_up(size_t v, size_t a) { return (v + a - 1) / a * a; }
-
-bool encode_2d(PrefillCtx* c, CUtensorMap* map, CUtensorMapDataType dt, const void* base, uint64_t inner, uint64_t rows,
-               uint64_t row_bytes, uint32_t box_rows) {
-    const cuuint64_t dims[2] = {inner, rows};
-    const cuuint64_t strides[1] = {row_bytes};
-    const cuuint32_t box[2] = {(cuuint32_t)PF_BK, box_rows};
-    const cuuint32_t estr[2] = {1, 1};
-    return c->encode(map, dt, 2, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
-                     CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
-}
-
 // the K half of one layer's pages as {d, token in page, kv head, k|v, page}; a box is 128 keys of one head
 bool encode_k_pages(PrefillCtx* c, CUtensorMap* map, CUtensorMapDataType dt, const void* base, int hd, int page_tokens, int kv_heads,
                     int num_pages) {
@@ -88,34 +72,6 @@ bool encode_k_pages(PrefillCtx* c, CUtensorMap* map, CUtensorMapDataType dt, con
     const cuuint32_t estr[5] = {1, 1, 1, 1, 1};
     return c->encode(map, dt, 5, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
                      CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
-}
-
-// instruction descriptor of tcgen05.mma kind::f16: fp32 accumulate, both operands K-major, M = 128
-inline uint32_t make_idesc(int bn, bool bf16) {
-    const uint32_t fmt = bf16 ? 1u : 0u;
-    return (1u << 4) | (fmt << 7) | (fmt << 10) | ((uint32_t)(bn >> 3) << 17) | ((uint32_t)(PF_BM >> 4) << 24);
-}
-
-template <int BN, bool SPLIT, class Epi>
-cudaError_t pf_launch_t(cd_model* m, const CUtensorMap& a, const CUtensorMap& a_lo, const CUtensorMap& b, const PfGemm& p, bool bf16, int zdim,
-                        const Epi& epi) {
-    auto kern = pf_gemm_kernel<BN, SPLIT, Epi>;
-    static bool attr_set = false;  // per instantiation
-    if (!attr_set) {
-        cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)PfTile<BN, SPLIT>::SMEM);
-        if (e != cudaSuccess) return e;
-        attr_set = true;
-    }
-    const dim3 grid((p.N + BN - 1) / BN, (p.M + PF_BM - 1) / PF_BM, zdim);
-    kern<<<grid, PF_THREADS, PfTile<BN, SPLIT>::SMEM, m->stream>>>(a, a_lo, b, p, make_idesc(BN, bf16), epi);
-    m->launches++;
-    return cudaGetLastError();
-}
-
-// a: the activation's hi and lo maps (lo unused when split is off)
-template <int BN, class Epi>
-cudaError_t pf_launch(cd_model* m, bool split, const CUtensorMap (&a)[2], const CUtensorMap& b, const PfGemm& p, bool bf16, int zdim, const Epi& epi) {
-    return split ? pf_launch_t<BN, true>(m, a[0], a[1], b, p, bf16, zdim, epi) : pf_launch_t<BN, false>(m, a[0], a[0], b, p, bf16, zdim, epi);
 }
 
 // the few-rows GEMM: w in 128-row boxes, x = the [NB][K] activation block (hi rows, then lo rows)
@@ -155,8 +111,8 @@ int ensure_weight_maps(cd_model* m, PrefillCtx* c, CUtensorMapDataType dt, CUten
     const int D = cf.dim, Q = cf.q_dim, KV = cf.kv_dim, H = cf.hidden;
     c->w_qkv.resize(cf.nlayers); c->w_o.resize(cf.nlayers); c->w_13.resize(cf.nlayers); c->w_2.resize(cf.nlayers); c->k_pages.resize(cf.nlayers);
     c->sk_qkv.resize(cf.nlayers); c->sk_o.resize(cf.nlayers); c->sk_13.resize(cf.nlayers); c->sk_2.resize(cf.nlayers);
-    bool ok = encode_2d(c, &c->w_head, dt, m->lm_head, D, m->v_loc, (uint64_t)D * 2, 256) &&
-              encode_2d(c, &c->sk_head, dt, m->lm_head, D, m->v_loc, (uint64_t)D * 2, 128);
+    bool ok = encode_2d(c->encode, &c->w_head, dt, m->lm_head, D, m->v_loc, (uint64_t)D * 2, 256) &&
+              encode_2d(c->encode, &c->sk_head, dt, m->lm_head, D, m->v_loc, (uint64_t)D * 2, 128);
     if (m->opt.weight_dtype == CD_DTYPE_FP8_E4M3) {
         const size_t n_qkv = (size_t)(Q + 2 * KV) * D, n_o = (size_t)D * Q, n_13 = (size_t)2 * H * D, n_2 = (size_t)D * H;
         if (cudaMalloc(&c->f8_qkv, n_qkv * 2) != cudaSuccess || cudaMalloc(&c->f8_o, n_o * 2) != cudaSuccess ||
@@ -165,10 +121,10 @@ int ensure_weight_maps(cd_model* m, PrefillCtx* c, CUtensorMapDataType dt, CUten
             return fail(m, CD_ERR_CUDA, "prompt-pass buffers for the widened FP8 matrices");
         }
         for (int l = 0; l < cf.nlayers && ok; ++l) {
-            ok = ok && encode_2d(c, &c->w_qkv[l], dt, c->f8_qkv, D, Q + 2 * KV, (uint64_t)D * 2, 256);
-            ok = ok && encode_2d(c, &c->w_o[l], dt, c->f8_o, Q, D, (uint64_t)Q * 2, 256);
-            ok = ok && encode_2d(c, &c->w_13[l], dt, c->f8_13, D, 2 * H, (uint64_t)D * 2, 256);
-            ok = ok && encode_2d(c, &c->w_2[l], dt, c->f8_2, H, D, (uint64_t)H * 2, 256);
+            ok = ok && encode_2d(c->encode, &c->w_qkv[l], dt, c->f8_qkv, D, Q + 2 * KV, (uint64_t)D * 2, 256);
+            ok = ok && encode_2d(c->encode, &c->w_o[l], dt, c->f8_o, Q, D, (uint64_t)Q * 2, 256);
+            ok = ok && encode_2d(c->encode, &c->w_13[l], dt, c->f8_13, D, 2 * H, (uint64_t)D * 2, 256);
+            ok = ok && encode_2d(c->encode, &c->w_2[l], dt, c->f8_2, H, D, (uint64_t)H * 2, 256);
             ok = ok && encode_k_pages(c, &c->k_pages[l], kdt, m->layers[l].kv, cf.hd, m->page_tokens, cf.kv_heads, m->num_pages);
         }
         if (!ok) { c->w_qkv.clear(); return fail(m, CD_ERR_CUDA, "cuTensorMapEncodeTiled failed for a weight matrix"); }
@@ -176,14 +132,14 @@ int ensure_weight_maps(cd_model* m, PrefillCtx* c, CUtensorMapDataType dt, CUten
     }
     for (int l = 0; l < cf.nlayers && ok; ++l) {
         const cd_layer_dev& L = m->layers[l];
-        ok = ok && encode_2d(c, &c->sk_qkv[l], dt, L.wqkv, D, Q + 2 * KV, (uint64_t)D * 2, 128);
-        ok = ok && encode_2d(c, &c->sk_o[l], dt, L.wo, Q, D, (uint64_t)Q * 2, 128);
-        ok = ok && encode_2d(c, &c->sk_13[l], dt, L.w13, D, 2 * H, (uint64_t)D * 2, 128);
-        ok = ok && encode_2d(c, &c->sk_2[l], dt, L.w2, H, D, (uint64_t)H * 2, 128);
-        ok = ok && encode_2d(c, &c->w_qkv[l], dt, L.wqkv, D, Q + 2 * KV, (uint64_t)D * 2, 256);
-        ok = ok && encode_2d(c, &c->w_o[l], dt, L.wo, Q, D, (uint64_t)Q * 2, 256);
-        ok = ok && encode_2d(c, &c->w_13[l], dt, L.w13, D, 2 * H, (uint64_t)D * 2, 256);
-        ok = ok && encode_2d(c, &c->w_2[l], dt, L.w2, H, D, (uint64_t)H * 2, 256);
+        ok = ok && encode_2d(c->encode, &c->sk_qkv[l], dt, L.wqkv, D, Q + 2 * KV, (uint64_t)D * 2, 128);
+        ok = ok && encode_2d(c->encode, &c->sk_o[l], dt, L.wo, Q, D, (uint64_t)Q * 2, 128);
+        ok = ok && encode_2d(c->encode, &c->sk_13[l], dt, L.w13, D, 2 * H, (uint64_t)D * 2, 128);
+        ok = ok && encode_2d(c->encode, &c->sk_2[l], dt, L.w2, H, D, (uint64_t)H * 2, 128);
+        ok = ok && encode_2d(c->encode, &c->w_qkv[l], dt, L.wqkv, D, Q + 2 * KV, (uint64_t)D * 2, 256);
+        ok = ok && encode_2d(c->encode, &c->w_o[l], dt, L.wo, Q, D, (uint64_t)Q * 2, 256);
+        ok = ok && encode_2d(c->encode, &c->w_13[l], dt, L.w13, D, 2 * H, (uint64_t)D * 2, 256);
+        ok = ok && encode_2d(c->encode, &c->w_2[l], dt, L.w2, H, D, (uint64_t)H * 2, 256);
         ok = ok && encode_k_pages(c, &c->k_pages[l], kdt, L.kv, cf.hd, m->page_tokens, cf.kv_heads, m->num_pages);
     }
     if (!ok) { c->w_qkv.clear(); return fail(m, CD_ERR_CUDA, "cuTensorMapEncodeTiled failed for a weight matrix"); }
@@ -202,13 +158,10 @@ int get_ctx(cd_model* m, PrefillCtx** out, bool fp8_ok, bool tp_ok = false) {
     PrefillCtx* c = (PrefillCtx*)m->prefill_ctx;
     if (!c) {
         c = new PrefillCtx();
-        void* fn = nullptr;
-        cudaDriverEntryPointQueryResult qres;
-        if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &fn, cudaEnableDefault, &qres) != cudaSuccess || qres != cudaDriverEntryPointSuccess || !fn) {
+        if (!(c->encode = encode_tiled_fn())) {
             delete c;
             return fail(m, CD_ERR_CUDA, "cuTensorMapEncodeTiled is not available from this driver");
         }
-        c->encode = (EncodeTiledFn)fn;
         m->prefill_ctx = c;
     }
     *out = c;
@@ -254,11 +207,11 @@ int run(cd_model* m, PrefillCtx* c, size_t n, bool split) {
     T16* gate_lo = split ? gate + R * (size_t)H : nullptr;
     KT* p_lo = split ? pm + (size_t)cf.heads * plane : nullptr;
     CUtensorMap a_xn[2], a_attn[2], a_gate[2], a_q[2], a_p[2], b_vt;
-    bool ok = encode_2d(c, &b_vt, kdt, c->vt, KL, (uint64_t)cf.kv_heads * hd, (uint64_t)KL * 2, (uint32_t)hd);
+    bool ok = encode_2d(c->encode, &b_vt, kdt, c->vt, KL, (uint64_t)cf.kv_heads * hd, (uint64_t)KL * 2, (uint32_t)hd);
     for (int h = 0; h < (split ? 2 : 1) && ok; ++h) {
-        ok = encode_2d(c, &a_xn[h], dt, h ? xn_lo : xn, D, R, (uint64_t)D * 2, PF_BM) && encode_2d(c, &a_attn[h], dt, h ? xn_lo : xn, Q, R, (uint64_t)Q * 2, PF_BM) &&
-             encode_2d(c, &a_gate[h], dt, h ? gate_lo : gate, H, R, (uint64_t)H * 2, PF_BM) && encode_2d(c, &a_q[h], kdt, h ? q_lo : qb, Q, R, (uint64_t)Q * 2, PF_BM) &&
-             encode_2d(c, &a_p[h], kdt, h ? p_lo : pm, KL, (uint64_t)cf.heads * R, (uint64_t)KL * 2, PF_BM);
+        ok = encode_2d(c->encode, &a_xn[h], dt, h ? xn_lo : xn, D, R, (uint64_t)D * 2, PF_BM) && encode_2d(c->encode, &a_attn[h], dt, h ? xn_lo : xn, Q, R, (uint64_t)Q * 2, PF_BM) &&
+             encode_2d(c->encode, &a_gate[h], dt, h ? gate_lo : gate, H, R, (uint64_t)H * 2, PF_BM) && encode_2d(c->encode, &a_q[h], kdt, h ? q_lo : qb, Q, R, (uint64_t)Q * 2, PF_BM) &&
+             encode_2d(c->encode, &a_p[h], kdt, h ? p_lo : pm, KL, (uint64_t)cf.heads * R, (uint64_t)KL * 2, PF_BM);
     }
     if (!ok) return fail(m, CD_ERR_CUDA, "cuTensorMapEncodeTiled failed for an activation buffer");
 
@@ -411,8 +364,8 @@ int run_samples(cd_model* m, PrefillCtx* c, const uint32_t* first, int ns, size_
     // one map per activation buffer: rows 0-15 the hi parts, rows 16-31 the lo parts
     const uint32_t xrows = split ? 2 * SK_ROWS : SK_ROWS;
     CUtensorMap a_xn, a_attn, a_gate;
-    const bool ok = encode_2d(c, &a_xn, dt, xn, D, xrows, (uint64_t)D * 2, xrows) && encode_2d(c, &a_attn, dt, xn, Q, xrows, (uint64_t)Q * 2, xrows) &&
-                    encode_2d(c, &a_gate, dt, gate, H, xrows, (uint64_t)H * 2, xrows);
+    const bool ok = encode_2d(c->encode, &a_xn, dt, xn, D, xrows, (uint64_t)D * 2, xrows) && encode_2d(c->encode, &a_attn, dt, xn, Q, xrows, (uint64_t)Q * 2, xrows) &&
+                    encode_2d(c->encode, &a_gate, dt, gate, H, xrows, (uint64_t)H * 2, xrows);
     if (!ok) return fail(m, CD_ERR_CUDA, "cuTensorMapEncodeTiled failed for an activation buffer");
 
     // page tables: prompt pages that are full are shared, the page the prompt ends in is copied, later pages are the sample's own
@@ -579,6 +532,10 @@ int prefill_batched(cd_model* m, size_t n) {
     if (dt == CD_DTYPE_F16) return run<__half, __half>(m, c, n, split);
     // bf16 and FP8 linears: bf16 activations and head; the cache is fp16 or bf16
     return m->kv_dtype == CD_DTYPE_F16 ? run<__nv_bfloat16, __half>(m, c, n, split) : run<__nv_bfloat16, __nv_bfloat16>(m, c, n, split);
+}
+
+const float* prefill_hidden_row(const cd_model* m, size_t i) {
+    return static_cast<const PrefillCtx*>(m->prefill_ctx)->x + i * (size_t)m->cfg.dim;
 }
 
 void prefill_release(cd_model* m) {

@@ -53,6 +53,10 @@ struct PfGemm {
     // row scale stored behind row n of the quantised matrix (Wfmt<Fp8Row>), nullptr otherwise
     const unsigned char* qrows;
     uint32_t qstride, qscale_off;
+    // grouped problem (a mixture of experts): row tile y multiplies the B rows of group tile_group[y], `group_rows` apart;
+    // a negative entry is a tile nobody needs.  nullptr: one matrix
+    const int* tile_group;
+    int group_rows;
 };
 
 // ------------------------------------------------------------------ PTX wrappers
@@ -238,6 +242,12 @@ pf_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant_
     extern __shared__ unsigned char pf_raw[];
     const int m0 = blockIdx.y * PF_BM, n0 = blockIdx.x * BN, z = blockIdx.z;
     if (p.causal == 1 && n0 > p.pos0 + m0 + PF_BM - 1) return;  // every key of this tile lies after every query of it
+    int b_row0 = n0;
+    if (p.tile_group != nullptr) {
+        const int g = p.tile_group[blockIdx.y];
+        if (g < 0) return;
+        b_row0 += g * p.group_rows;
+    }
     int kmax = p.K;
     if (p.causal == 2) kmax = min(kmax, p.pos0 + m0 + PF_BM);    // P is zero beyond the diagonal
     const int nkb = (kmax + PF_BK - 1) / PF_BK;
@@ -278,7 +288,7 @@ pf_gemm_kernel(const __grid_constant__ CUtensorMap tma_a, const __grid_constant_
                 tma_load_2d(a_dst, &tma_a, z * p.a_col_z + kb * PF_BK, z * p.a_row_z + m0, full0 + 8u * s);
                 if (SPLIT) tma_load_2d(a_dst + TL::A_BYTES, &tma_a_lo, z * p.a_col_z + kb * PF_BK, z * p.a_row_z + m0, full0 + 8u * s);
                 if (p.b_paged) tma_load_5d(b_dst, &tma_b, kb * PF_BK, 0, zb, 0, n0 / p.page_tokens, full0 + 8u * s);
-                else tma_load_2d(b_dst, &tma_b, kb * PF_BK, zb * p.b_row_z + n0, full0 + 8u * s);
+                else tma_load_2d(b_dst, &tma_b, kb * PF_BK, zb * p.b_row_z + b_row0, full0 + 8u * s);
             }
         }
     } else if (warp == 1) {

@@ -84,7 +84,7 @@ int restore_base(cd_session* s) {
     const uint32_t* w;
     size_t n;
     window_of(s->prompt_ids, (size_t)s->cfg.seq, &w, &n);
-    if (s->cache_tokens.size() >= n && std::equal(w, w + n, s->cache_tokens.begin())) return CD_OK;
+    if (s->cache_tokens.size() >= n && std::equal(w, w + n, s->cache_tokens.begin()) && cd_can_rewind(s->m, n)) return CD_OK;
     std::vector<float> scratch(s->cfg.vocab);
     return full_forward(s, s->prompt_ids, scratch.data());
 }
