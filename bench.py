@@ -266,6 +266,127 @@ def bench_moe(R, np, local_rank, rank, world, use_graph):
             "token_roofline_frac_of_measured_peak": moe_bytes_per_token(MOE_PROMPT + MOE_STEPS / 2) / world * rate1 / 1e9 / peak}
 
 
+def dafidra_config(width, layers, vocab, heads, kv_heads, head, window, mem_heads, mem_dim, mem_vdim, mlp):
+    """A Dafidra configuration with the same layer everywhere, at a real model's widths."""
+    layer = {"type": "parallel", "mlp": mlp, "mixer": {
+        "left": {"heads": heads, "kv_heads": kv_heads, "dim": head, "vdim": head, "scale": head ** -0.5, "mask": {"size": window}, "q_temp": {"coef": 0.1, "every": 4096}},
+        "right": {"heads": mem_heads, "dim": mem_dim, "vdim": mem_vdim, "gate_cap": 15.0}}}
+    return {"architecture": "Dafidra", "width": width, "vocab": vocab, "norm": {"eps": 1e-5}, "residual_mult": 0.5, "layers": [layer] * layers}
+
+
+# name -> (Dafidra configuration, the closest existing model at equal width, depth, vocabulary and active FFN columns)
+DAFIDRA_SIZES = {
+    "1b_dense": (dafidra_config(2048, 24, 32000, 16, 4, 128, 1024, 8, 128, 256, {"kind": "dense", "ff": 5632}),
+                 ("dense", dict(dim=2048, hidden=5632, heads=16, kv_heads=4, hd=128, seq=8192, nlayers=24, vocab=32000))),
+    "5b_dense": (dafidra_config(4096, 26, 32000, 32, 8, 128, 1024, 16, 128, 256, {"kind": "dense", "ff": 11008}),
+                 ("dense", dict(dim=4096, hidden=11008, heads=32, kv_heads=8, hd=128, seq=8192, nlayers=26, vocab=32000))),
+    "moe": (dafidra_config(2048, 24, 32000, 16, 4, 128, 1024, 8, 128, 256,
+                           {"kind": "moe", "expert": {"ff": 1408}, "router": {"experts": 64, "top": 8, "groups": {"count": 8, "keep": 4}}}),
+            ("moe_mla", MOE)),
+}
+
+
+def dafidra_bytes(cfg, ctx):
+    """Algorithmic HBM bytes of one decoded token by kernel class (bf16 weights, fp16 cache, fp32 state read and written)."""
+    D, out = cfg["width"], dict.fromkeys(("qkv_gemv", "attention", "wo_gemv", "w13_gemv", "w2_gemv"), 0)
+    for L in cfg["layers"]:
+        a, r, f = L["mixer"]["left"], L["mixer"]["right"], L["mlp"]
+        rows = a["heads"] * a["dim"] + a["kv_heads"] * (a["dim"] + a["vdim"]) + a["heads"] + r["heads"] * (2 * r["dim"] + 2 * r["vdim"] + 2)
+        out["qkv_gemv"] += rows * D * 2
+        out["attention"] += min(a["mask"]["size"], ctx) * a["kv_heads"] * (a["dim"] + a["vdim"]) * 2 + 2 * 4 * r["heads"] * r["dim"] * r["vdim"]
+        out["wo_gemv"] += D * (a["heads"] * a["vdim"] + r["heads"] * r["vdim"]) * 2
+        if f["kind"] == "dense":
+            cols, extra = f["ff"], 0
+        else:
+            cols, extra = f["expert"]["ff"] * f["router"]["top"], f["router"]["experts"] * D * 2
+        out["w13_gemv"] += 2 * cols * D * 2 + extra
+        out["w2_gemv"] += cols * D * 2
+    out["head_gemv"] = cfg["vocab"] * D * 2
+    return out
+
+
+def existing_bytes(kind, c, ctx):
+    """The same for the dense family and for the MoE + MLA decoder."""
+    D, L = (c["dim"], c["nlayers"])
+    if kind == "dense":
+        Q, KV, H = c["heads"] * c["hd"], c["kv_heads"] * c["hd"], c["hidden"]
+        out = {"qkv_gemv": D * (Q + 2 * KV) * 2, "attention": 2 * ctx * KV * 2, "wo_gemv": D * Q * 2, "w13_gemv": 2 * H * D * 2, "w2_gemv": H * D * 2}
+    else:
+        qh, w, n = c["nope_dim"] + c["rope_dim"], c["kv_latent"] + c["rope_dim"], c["top_k"] + c["n_shared"]
+        out = {"qkv_gemv": D * (c["heads"] * qh + w) * 2, "attention": ctx * w * 2 + c["kv_latent"] * c["heads"] * (c["nope_dim"] + c["v_dim"]) * 2,
+               "wo_gemv": c["heads"] * c["v_dim"] * D * 2, "w13_gemv": 2 * n * c["hidden"] * D * 2 + c["n_experts"] * D * 2, "w2_gemv": n * c["hidden"] * D * 2}
+    out = {k: v * L for k, v in out.items()}
+    out["head_gemv"] = c["vocab"] * D * 2
+    return out
+
+
+def bench_dafidra(sizes):
+    """Prefill and decode throughput of the Dafidra decoder (random weights) beside the closest existing family at equal
+    size, with the time and roofline fraction of every kernel class of one token.  Prints one JSON line per size."""
+    import numpy as np
+
+    import rustane_b200 as R
+    peak, kind = measured_peak_gbs()
+    ctx, steps = 2048, 128
+
+    def measure(model, vocab, by_class, prompts):
+        out = {}
+        for n in prompts:
+            ids = R.synth_prompt(3, vocab, n)
+            for _ in range(3):
+                model.set_len(0)
+                model.prefill(ids)
+            out["prefill%d_tokens_per_s" % n] = n / (model.last_device_ms() / 1e3)
+        model.set_len(0)
+        logits = model.prefill(R.synth_prompt(3, vocab, ctx))
+        first = int(np.argmax(logits))
+        for _ in range(3):
+            model.set_len(ctx)
+            ids = model.decode_steps_greedy(first, steps)
+        total = sum(by_class.values())
+        out["decode_tokens_per_s"] = steps / (model.last_device_ms() / 1e3)
+        out["hbm_bytes_per_token"] = total
+        out["token_roofline_frac"] = total * out["decode_tokens_per_s"] / 1e9 / peak
+        model.set_len(ctx)
+        model.profile_decode_step(int(ids[0]))
+        model.set_len(ctx)
+        prof = model.profile_decode_step(int(ids[0]))
+        out["classes"] = {k: {"ms": round(prof[k][0], 4), "launches": prof[k][1], "roofline_frac": round(by_class[k] / (prof[k][0] / 1e3) / 1e9 / peak, 4)}
+                          for k in by_class if prof[k][0] > 0}
+        model.close()
+        return out
+
+    for name in sizes:
+        cfg, (closest, dims) = DAFIDRA_SIZES[name]
+        line = {"size": name, "hbm_peak_gbs": peak, "peak_source": kind, "context": ctx, "decode_steps": steps,
+                "l2": "weights larger than L2 stream from HBM for every token and prompt pass", "data": "synthetic", "dtype": "bf16"}
+        sampler = ClockSampler(0)
+        sampler.start()
+        line["dafidra"] = measure(R.Model.from_config(cfg, 7, max_tokens=8192, use_graph=True), cfg["vocab"], dafidra_bytes(cfg, ctx), (1024, 2048, 4096))
+        if closest == "dense":
+            for label, mega in (("dense_per_operator", False), ("dense", True)):
+                line[label] = measure(R.Model.synthetic(R.Config(**dims), 7, dtype="bf16", use_graph=True, mega=mega), dims["vocab"], existing_bytes(closest, dims, ctx),
+                                      (1024, 2048, 4096))
+        else:
+            line[closest] = measure(R.Model.moe_synthetic(R.MoeConfig(**dims), 7, dtype="bf16", use_graph=True), dims["vocab"], existing_bytes(closest, dims, ctx), ())
+        line["clocks"] = sampler.stop()
+        print(json.dumps(line), flush=True)
+
+
+def profile_dafidra(size, prompt):
+    """Small case for `ncu` on the Dafidra decoder: two layers of one of the sizes; a prompt pass, then eight tokens."""
+    import rustane_b200 as R
+    cfg = dict(DAFIDRA_SIZES[size][0])
+    cfg["layers"] = cfg["layers"][:2]
+    model = R.Model.from_config(cfg, 7, max_tokens=8192)
+    for _ in range(2):
+        model.set_len(0)
+        model.prefill(R.synth_prompt(3, cfg["vocab"], prompt))
+    ms = model.last_device_ms()
+    model.decode_steps_greedy(1, 8)
+    print("Dafidra profile case done: %d launches, prompt pass %.3f ms, %.3f ms/token" % (model.kernel_launches(), ms, model.last_device_ms() / 8))
+
+
 def profile_case(dtype="bf16", per_operator=False):
     """Small case for `ncu`: identical kernels and shapes per layer, 3 of 26 layers (about
     1.5 GB resident, weights still far larger than L2), context 1024 (cache contents are
@@ -338,7 +459,15 @@ def main():
                     help="small case for ncu captures of the batched prompt pass (3 layers, 512 tokens); prints no bench line")
     ap.add_argument("--profile-samples", action="store_true",
                     help="small case for ncu captures of the multi-sample decode step (3 layers, 8 samples); prints no bench line")
+    ap.add_argument("--dafidra", nargs="*", choices=sorted(DAFIDRA_SIZES), default=None,
+                    help="prefill and decode throughput of the Dafidra decoder beside the closest existing family (all sizes, or the named ones)")
+    ap.add_argument("--profile-dafidra", choices=sorted(DAFIDRA_SIZES), default=None,
+                    help="small case for ncu captures of the Dafidra decoder (two layers of a size, a 2048-token prompt, 8 tokens); prints no bench line")
     args = ap.parse_args()
+    if args.dafidra is not None:
+        return bench_dafidra(args.dafidra or sorted(DAFIDRA_SIZES))
+    if args.profile_dafidra:
+        return profile_dafidra(args.profile_dafidra, 2048)
     if args.profile_case:
         return profile_case(args.dtype, args.per_operator)
     if args.profile_moe:

@@ -46,9 +46,10 @@ def head_slopes(heads):
     return 2.0 ** (-8.0 * (np.arange(heads) + 1.0) / heads)
 
 
-def attention(h, W, p, c, eps, fault=""):
+def attention(h, W, p, c, eps, fault="", cache=None):
     """Windowed softmax attention: whole-projection q/k norm, temperature on q, linear distance bias, a sink in the
-    denominator, one output gate per head.  h [T, width] -> [T, width]."""
+    denominator, one output gate per head.  h [T, width] -> [T, width].  `cache` (a numpy type) rounds keys and values to
+    what a cache of that type holds."""
     T = h.shape[0]
     H, G, dim, vdim = c["heads"], c["kv_heads"], c["dim"], c["vdim"]
     q, k, v = h @ W[p + "q"].T, h @ W[p + "k"].T, h @ W[p + "v"].T
@@ -57,6 +58,8 @@ def attention(h, W, p, c, eps, fault=""):
     else:
         q = norm_plain(q, W[p + "q.norm"], eps)
     k = norm_plain(k, W[p + "k.norm"], eps)
+    if cache is not None:
+        k, v = k.astype(cache).astype(np.float64), v.astype(cache).astype(np.float64)
     pos = np.arange(T)
     if fault != "no_temperature":
         q = q * query_temperature(pos, c["q_temp"]["every"], c["q_temp"]["coef"])[:, None]
@@ -115,9 +118,9 @@ def matrix_memory(h, W, p, c, eps, fault="", state=None):
     return out @ W[p + "o"].T
 
 
-def parallel_mixer(h, W, p, c, eps, fault="", state=None):
+def parallel_mixer(h, W, p, c, eps, fault="", state=None, cache=None):
     """Both mixers on the same input, each output normed over the width, averaged."""
-    a = norm_plain(attention(h, W, p + "left.", c["left"], eps, fault), W[p + "left.out"], eps)
+    a = norm_plain(attention(h, W, p + "left.", c["left"], eps, fault, cache), W[p + "left.out"], eps)
     b = norm_plain(matrix_memory(h, W, p + "right.", c["right"], eps, fault, state), W[p + "right.out"], eps)
     return (a + b) * 0.5
 
@@ -144,7 +147,25 @@ def route(z, experts, top, groups=None, fault=""):
     return ranked, w
 
 
-def feed_forward(h, W, p, c, fault=""):
+def route_margin(z, experts, top, groups=None):
+    """How far a token's routing is from another outcome: the smallest relative gap between the scores (of experts, and of
+    groups) on either side of a choice."""
+    s = np.exp(z - z.max())
+    s = s / s.sum()
+    margin, allowed = 1.0, np.ones(experts, bool)
+    if groups and groups["keep"] < groups["count"]:
+        best = s.reshape(groups["count"], -1).max(axis=1)
+        r = np.sort(best)[::-1]
+        margin = min(margin, (r[groups["keep"] - 1] - r[groups["keep"]]) / r[groups["keep"] - 1])
+        kept = np.argsort(-best, kind="stable")[:groups["keep"]]
+        allowed = np.isin(np.arange(experts) // (experts // groups["count"]), kept)
+    r = np.sort(s[allowed])[::-1]
+    if top < len(r):
+        margin = min(margin, (r[top - 1] - r[top]) / r[top - 1])
+    return margin
+
+
+def feed_forward(h, W, p, c, fault="", margins=None):
     if c["kind"] == "dense":
         return gated_ffn(h, W, p)
     r = c["router"]
@@ -152,21 +173,24 @@ def feed_forward(h, W, p, c, fault=""):
     z = h @ W[p + "router"].T
     for t in range(h.shape[0]):
         ids, w = route(z[t], r["experts"], r["top"], r.get("groups"), fault)
+        if margins is not None:
+            margins.append(route_margin(z[t], r["experts"], r["top"], r.get("groups")))
         for e, we in zip(ids, w):
             out[t] += we * gated_ffn(h[t:t + 1], W, "%se%d." % (p, e))[0]
     return out
 
 
-def forward(cfg, W, tokens, fault="", taps=None):
-    """Logits [T, vocab] of a whole sequence.  `taps`, a list, receives the residual stream after every layer."""
+def forward(cfg, W, tokens, fault="", taps=None, margins=None, cache=None):
+    """Logits [T, vocab] of a whole sequence.  `taps`, a list, receives the residual stream after every layer, `margins`
+    the routing margin of every token and layer."""
     eps, mult = cfg["norm"]["eps"], cfg["residual_mult"]
     x = W["embed"][np.asarray(tokens)]
     for i, L in enumerate(cfg["layers"]):
         p = "l%d." % i
         assert L["type"] == "parallel"
-        x = x + mult * norm_around_zero(parallel_mixer(x, W, p + "mix.", L["mixer"], eps, fault), W[p + "norm1"], eps)
+        x = x + mult * norm_around_zero(parallel_mixer(x, W, p + "mix.", L["mixer"], eps, fault, cache=cache), W[p + "norm1"], eps)
         if L.get("mlp"):
-            x = x + mult * norm_around_zero(feed_forward(x, W, p + "mlp.", L["mlp"], fault), W[p + "norm2"], eps)
+            x = x + mult * norm_around_zero(feed_forward(x, W, p + "mlp.", L["mlp"], fault, margins), W[p + "norm2"], eps)
         if taps is not None:
             taps.append(x.copy())
     return norm_around_zero(x, W["final.norm"], eps) @ W["head"].T

@@ -79,6 +79,7 @@ SIGNATURES = {
     "cd_last_error": (C.c_char_p, [_vp]),
     "cd_len": (C.c_int, [_vp, _szp]),
     "cd_set_len": (C.c_int, [_vp, C.c_size_t]),
+    "cd_can_rewind": (C.c_int, [_vp, C.c_size_t]),
     "cd_seed_layer_cache_cf": (C.c_int, [_vp, C.c_int, C.c_size_t, _f32p, _f32p]),
     "cd_decode_token": (C.c_int, [_vp, _f32p, _f32p]),
     "cd_decode_token_from_id": (C.c_int, [_vp, C.c_uint32, _f32p]),
@@ -90,6 +91,9 @@ SIGNATURES = {
     "cd_materialize_current_logits_block": (C.c_int, [_vp, C.c_size_t, C.c_float, _f32p, C.c_size_t, _szp]),
     "cd_model_create_from_checkpoint": (C.c_int, [C.c_char_p, _P(CdOptions), _P(CdConfig), _vpp]),
     "cd_checkpoint_info": (C.c_int, [C.c_char_p, _P(CdConfig), _P(C.c_int32)]),
+    "cd_model_create_from_dir": (C.c_int, [C.c_char_p, C.c_size_t, _P(CdOptions), _vpp]),
+    "cd_model_create_from_config": (C.c_int, [C.c_char_p, C.c_size_t, _P(CdOptions), C.c_uint64, C.c_float, _vpp]),
+    "cd_config_info": (C.c_int, [C.c_char_p, _P(CdConfig)]),
     "cd_model_create_synthetic": (C.c_int, [_P(CdConfig), _P(CdOptions), C.c_uint64, C.c_float, C.c_int, _vpp]),
     "cd_synth_value": (C.c_float, [C.c_uint64, C.c_uint64, C.c_uint64, C.c_float]),
     "cd_synth_prompt": (None, [C.c_uint64, C.c_int, _u32p, C.c_int]),
@@ -109,6 +113,7 @@ SIGNATURES = {
     "cd_tp_connect_ptrs": (C.c_int, [_vp, _vpp, C.c_int]),
     "cd_decode_token_logits_from_id": (C.c_int, [_vp, C.c_uint32, C.c_float, _f32p]),
     "cd_prefill": (C.c_int, [_vp, _u32p, C.c_size_t, C.c_float, _f32p]),
+    "cd_prefill_logits": (C.c_int, [_vp, _u32p, C.c_size_t, _szp, C.c_size_t, C.c_float, _f32p]),
     "cd_decode_steps_greedy": (C.c_int, [_vp, C.c_uint32, C.c_size_t, _u32p]),
     "cd_decode_steps_topk": (C.c_int, [_vp, C.c_uint32, C.c_size_t, C.c_size_t, C.c_float, C.c_float, _u64p, _u32p]),
     "cd_decode_steps_fullvocab": (C.c_int, [_vp, C.c_uint32, C.c_size_t, C.c_float, C.c_float, _u64p, _u32p]),

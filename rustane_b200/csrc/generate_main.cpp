@@ -22,6 +22,8 @@ namespace {
 
 struct Args {
     std::string checkpoint;
+    std::string model_dir;   // a model folder (config.json + model.safetensors) instead of an RSTK checkpoint
+    long max_tokens = 0;     // its longest sequence (0: 4096)
     std::vector<uint32_t> prompt_ids;
     bool have_ids = false;
     int backend = CD_BACKEND_AUTO;
@@ -42,6 +44,7 @@ struct Args {
             "Usage: generate --checkpoint PATH --prompt-ids 1,2,3 [--decode-backend auto|naive|cuda] [--kv-cache] "
             "[--steps N] [--temperature T] [--top-k K] [--softcap S] [--samples N] [--seed N] [--jsonl-session] "
             "[--dtype f32|f16|bf16|fp8|int4] [--no-graph]\n"
+            "       generate --model DIR [--max-tokens N] ...                      (a folder with config.json and model.safetensors; same options)\n"
             "       generate --checkpoint PATH --convert-to OUT --dtype fp8|int4   (quantise the linears once; OUT loads without conversion)\n");
     exit(code);
 }
@@ -72,6 +75,8 @@ Args parse_args(int argc, char** argv) {
     for (int i = 1; i < argc;) {
         const std::string k = argv[i];
         if (k == "--checkpoint") { a.checkpoint = need(i); i += 2; }
+        else if (k == "--model") { a.model_dir = need(i); i += 2; }
+        else if (k == "--max-tokens") { a.max_tokens = atol(need(i).c_str()); i += 2; }
         else if (k == "--prompt-ids") { if (!parse_ids(need(i), &a.prompt_ids)) die("prompt ids must be integers"); a.have_ids = true; i += 2; }
         else if (k == "--prompt" || k == "--tokenizer") die("text prompts need a tokenizer, which this build does not include; pass --prompt-ids");
         else if (k == "--add-special-tokens" || k == "--no-skip-special-tokens") i += 1;
@@ -99,7 +104,8 @@ Args parse_args(int argc, char** argv) {
     if (a.prompt_ids.empty()) die("--prompt-ids must contain at least one token id");
     if (a.samples <= 0) die("--samples must be >= 1");
     if (a.steps < 0) die("--steps must be an integer");
-    if (a.checkpoint.empty()) { fprintf(stderr, "--checkpoint required\n"); usage(1); }
+    if (a.checkpoint.empty() == a.model_dir.empty()) { fprintf(stderr, "pass one of --checkpoint and --model\n"); usage(1); }
+    if (a.max_tokens < 0) die("--max-tokens must not be negative");
     return a;
 }
 
@@ -303,11 +309,15 @@ int main(int argc, char** argv) {
     if (opts.weight_dtype == -2) die("--dtype must be one of: f32, f16, bf16, fp8, int4");
     cd_config cfg;
     int32_t meta[4] = {0, 0, 0, 0};
-    if (cd_checkpoint_info(args.checkpoint.c_str(), &cfg, meta)) die(std::string("failed to load checkpoint: ") + cd_last_error(nullptr));
+    const bool folder = !args.model_dir.empty();
+    if (!folder && cd_checkpoint_info(args.checkpoint.c_str(), &cfg, meta)) die(std::string("failed to load checkpoint: ") + cd_last_error(nullptr));
     const auto t_load = std::chrono::steady_clock::now();
     cd_model* model = nullptr;
-    if (cd_model_create_from_checkpoint(args.checkpoint.c_str(), &opts, &cfg, &model))
+    const int rc_load = folder ? cd_model_create_from_dir(args.model_dir.c_str(), (size_t)args.max_tokens, &opts, &model)
+                               : cd_model_create_from_checkpoint(args.checkpoint.c_str(), &opts, &cfg, &model);
+    if (rc_load)
         die(std::string("failed to load checkpoint: ") + cd_last_error(nullptr));
+    if (folder) cd_model_get_config(model, &cfg, nullptr, nullptr);
     const double load_s = std::chrono::duration<double>(std::chrono::steady_clock::now() - t_load).count();
 
     const size_t eff_ctx = std::min(args.prompt_ids.size(), (size_t)cfg.seq);

@@ -259,6 +259,7 @@ __device__ inline void mem_step(const MixerStep& p, int idx, float* sm, float* r
     const float m0 = __ldcg(mrun), mt = fmaxf(gf + m0, gi), fa = expf(gf + m0 - mt), ia = expf(gi - mt);
     const float qscale = 1.0f / sqrtf((float)d.dim);
     float nq = 0.0f;
+#pragma unroll 2
     for (int i = tid; i < d.dim; i += MIX_THREADS) {
         const float q = __ldcg(p.proj + p.pl.rq + h * d.dim + i) * qscale, k = __ldcg(p.proj + p.pl.rk + h * d.dim + i);
         qs[i] = q;
@@ -342,8 +343,10 @@ __device__ inline void attn_step(const MixerStep& p, KT* __restrict__ pool, int 
     if (t0 < t1) {
         float sq = 0.0f, sk = 0.0f;
         const bool newest = t1 == pos + 1;  // this slice holds the current position
+#pragma unroll 8
         for (int i = tid; i < a.H * a.dim; i += MIX_THREADS) { const float v = __ldcg(p.proj + p.pl.lq + i); sq = fmaf(v, v, sq); }
         if (newest)
+#pragma unroll 4
             for (int i = tid; i < a.G * a.dim; i += MIX_THREADS) { const float v = __ldcg(p.proj + p.pl.lk + i); sk = fmaf(v, v, sk); }
         const float rq = a.temperature(pos) * a.scale / sqrtf(block_sum(sq, red) / (float)(a.H * a.dim) + a.eps);
         for (int i = tid; i < a.kp; i += MIX_THREADS)

@@ -632,25 +632,34 @@ struct RouterMixIn {  // the residual stream behind two parallel mixers (InParal
     const float *x, *yl, *yr, *wl, *wr, *gain;
     float* out;
     float mult, eps;
-    __device__ float fill(float* xs, float* red, int dim, bool writer) const {
+    __device__ float fill(float* xs, float* red, int dim, bool writer) const {  // dim is a multiple of 4
+        const int n4 = dim / 4, step = blockDim.x;
+        auto at = [](const float* p, int i) { return __ldcg(reinterpret_cast<const float4*>(p) + i); };
+        auto weight = [](const float* p, int i) { return reinterpret_cast<const float4*>(p)[i]; };
+        float4* x4 = reinterpret_cast<float4*>(xs);
         float sl = 0.0f, sr = 0.0f, ss = 0.0f;
-        for (int i = threadIdx.x; i < dim; i += blockDim.x) {
-            const float a = __ldcg(yl + i), b = __ldcg(yr + i);
-            sl = fmaf(a, a, sl);
-            sr = fmaf(b, b, sr);
+#pragma unroll 4
+        for (int i = threadIdx.x; i < n4; i += step) {
+            const float4 a = at(yl, i), b = at(yr, i);
+            sl += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+            sr += b.x * b.x + b.y * b.y + b.z * b.z + b.w * b.w;
         }
         const float rl = 0.5f / sqrtf(block_sum(sl, red) * (1.0f / (float)dim) + eps);
         const float rr = 0.5f / sqrtf(block_sum(sr, red) * (1.0f / (float)dim) + eps);
-        for (int i = threadIdx.x; i < dim; i += blockDim.x) {
-            const float z = __ldcg(yl + i) * rl * wl[i] + __ldcg(yr + i) * rr * wr[i];
-            xs[i] = z;
-            ss = fmaf(z, z, ss);
+#pragma unroll 4
+        for (int i = threadIdx.x; i < n4; i += step) {
+            const float4 a = at(yl, i), b = at(yr, i), p = weight(wl, i), q = weight(wr, i);
+            const float4 z = make_float4(a.x * rl * p.x + b.x * rr * q.x, a.y * rl * p.y + b.y * rr * q.y, a.z * rl * p.z + b.z * rr * q.z, a.w * rl * p.w + b.w * rr * q.w);
+            x4[i] = z;
+            ss += z.x * z.x + z.y * z.y + z.z * z.z + z.w * z.w;
         }
         const float r = mult / sqrtf(block_sum(ss, red) * (1.0f / (float)dim) + eps);
-        for (int i = threadIdx.x; i < dim; i += blockDim.x) {
-            const float v = __ldcg(x + i) + xs[i] * r * gain[i];
-            xs[i] = v;
-            if (writer) out[i] = v;
+#pragma unroll 4
+        for (int i = threadIdx.x; i < n4; i += step) {
+            const float4 b = at(x, i), g = weight(gain, i), z = x4[i];
+            const float4 v = make_float4(b.x + z.x * r * g.x, b.y + z.y * r * g.y, b.z + z.z * r * g.z, b.w + z.w * r * g.w);
+            x4[i] = v;
+            if (writer) reinterpret_cast<float4*>(out)[i] = v;
         }
         __syncthreads();
         return 1.0f;
@@ -666,7 +675,7 @@ __global__ void __launch_bounds__(128)
 moe_router_kernel(In in, const WT* __restrict__ wr, float* __restrict__ logits, unsigned int* __restrict__ counter, int* __restrict__ sel_ids,
                   float* __restrict__ sel_w, int* __restrict__ loc_ids, float* __restrict__ loc_w, int* __restrict__ n_loc, int dim, RouteRule rule,
                   int e0, int n_local) {
-    extern __shared__ float sm[];  // [dim] the input; the last CTA: [experts] scores and [groups] on top of it
+    extern __shared__ __align__(16) float sm[];  // [dim] the input; the last CTA: [experts] scores and [groups] on top of it
     __shared__ float red[32];
     __shared__ int s_last;
     constexpr int EPC = Elem<WT>::EPC, PRE = 8;

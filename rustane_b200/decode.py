@@ -5,6 +5,7 @@ Method names, argument meaning and error behaviour follow the reference; where t
 reference panics (assert!/expect) these raise CudaDecodeError carrying the same message.
 """
 import ctypes as C
+import json
 import os
 
 import numpy as np
@@ -162,6 +163,33 @@ class Model:
             raise CudaDecodeError(rc, lib.cd_last_error(None).decode())
         return cls(h.value, Config.from_c(c))
 
+    @classmethod
+    def _configured(cls, h):
+        c = _ffi.CdConfig()
+        lib.cd_model_get_config(h, C.byref(c), None, None)
+        return cls(h.value, Config.from_c(c))
+
+    @classmethod
+    def from_pretrained(cls, path, max_tokens=0, dtype=None, **opts):
+        """A model folder: config.json (its "architecture" picks the registered reader) and model.safetensors.
+        max_tokens (0: 4096) bounds the sequence; dtype "bf16" (default) or "f32"."""
+        o, h = _options(**opts), C.c_void_p()
+        o.weight_dtype = -1 if dtype is None else _DTYPES[dtype]
+        rc = lib.cd_model_create_from_dir(os.fsencode(path), max_tokens, C.byref(o), C.byref(h))
+        if rc:
+            raise CudaDecodeError(rc, lib.cd_last_error(None).decode())
+        return cls._configured(h)
+
+    @classmethod
+    def from_config(cls, config, seed, std=0.02, max_tokens=0, dtype=None, **opts):
+        """The same from a configuration (a dict) with seeded synthetic weights."""
+        o, h = _options(**opts), C.c_void_p()
+        o.weight_dtype = -1 if dtype is None else _DTYPES[dtype]
+        rc = lib.cd_model_create_from_config(json.dumps(config).encode(), max_tokens, C.byref(o), seed, std, C.byref(h))
+        if rc:
+            raise CudaDecodeError(rc, lib.cd_last_error(None).decode())
+        return cls._configured(h)
+
     def save_quantised(self, path):
         """Write this (single-GPU, dense, FP8 or INT4) model as a quantised RSTK v3 file."""
         self._check(lib.cd_model_save_quantised(self._h, os.fsencode(path)))
@@ -192,6 +220,10 @@ class Model:
 
     def set_len(self, n):
         self._check(lib.cd_set_len(self._h, n))
+
+    def can_rewind(self, n):
+        """Whether set_len(n) would succeed (a family with recurrent state keeps it at a few lengths only)."""
+        return bool(lib.cd_can_rewind(self._h, n))
 
     def seed_layer_cache_from_channel_first(self, layer_idx, live_len, k_rope_cf, v_cf):
         k, v = _cf32(k_rope_cf), _cf32(v_cf)
@@ -260,6 +292,14 @@ class Model:
         ids = np.ascontiguousarray(ids, dtype=np.uint32)
         out = np.empty(self.cfg.vocab, dtype=np.float32) if want_logits else None
         self._check(lib.cd_prefill(self._h, _u32(ids), len(ids), softcap, _f32(out) if want_logits else None))
+        return out
+
+    def prefill_logits(self, ids, want, softcap=0.0):
+        """Feed `ids` behind the cached tokens; logits [len(want), vocab] at the places `want` among them."""
+        ids = np.ascontiguousarray(ids, dtype=np.uint32)
+        places = (C.c_size_t * max(len(want), 1))(*[int(w) for w in want])
+        out = np.empty((len(want), self.cfg.vocab), dtype=np.float32)
+        self._check(lib.cd_prefill_logits(self._h, _u32(ids), len(ids), places, len(want), softcap, _f32(out)))
         return out
 
     def decode_steps_greedy(self, first_token, nsteps):
@@ -344,6 +384,15 @@ class Model:
         n = C.c_uint64()
         self._check(lib.cd_kernel_launches(self._h, C.byref(n)))
         return n.value
+
+
+def config_info(config):
+    """Parse and validate a configured architecture's config (a dict or JSON text) on the host; raises ValueError."""
+    text = config if isinstance(config, str) else json.dumps(config)
+    c = _ffi.CdConfig()
+    if lib.cd_config_info(text.encode(), C.byref(c)):
+        raise ValueError(lib.cd_last_error(None).decode())
+    return Config.from_c(c)
 
 
 def merge_topk_candidates(vals, idxs, top_k):
