@@ -52,8 +52,17 @@ cudaError_t hybrid_step_t(cd_model* m, const cd_step& p) {
     float *yl = S.y, *yr = S.y + D;
     auto ffn_in = [&](const cd_hybrid_layer& L) { return InNormedResidual{x[cur], S.y2, L.gain2, x[cur ^ 1], mult, eps, D}; };
     auto mix_in = [&](const cd_hybrid_layer& L) { return InParallelMix{x[cur], yl, yr, L.out_l, L.out_r, L.gain1, x[cur ^ 1], mult, eps, D}; };
+    // the next GEMV's first rows, pulled into L2 behind a GEMV's own last loads
+    auto hint = [&](const void* w, int K, int N, int unit) {
+        m->next_stream = NextStream{m->prefetch_kb > 0 ? w : nullptr, Wfmt<WT>::row_stride(K), N / unit, unit, (uint32_t)m->prefetch_kb * 1024u};
+    };
     for (int l = 0; l < c.nlayers; ++l) {
         const cd_hybrid_layer& L = S.layers[l];
+        const cd_hybrid_layer* next = l + 1 < c.nlayers ? &S.layers[l + 1] : nullptr;
+        auto hint_next = [&]() {
+            if (next) hint(next->wmix, D, next->proj.rows, 1);
+            else if (p.head != HEAD_NONE) hint(m->lm_head, D, m->v_loc, 1);
+        };
         m->cur_cls = CLS_QKV;
         const EpiStore to_proj{S.proj};
         if (!behind) {
@@ -84,15 +93,19 @@ cudaError_t hybrid_step_t(cd_model* m, const cd_step& p) {
         }
         m->cur_cls = CLS_WO;
         {
+            if (L.cfg.mlp.kind == FfnCfg::DENSE) hint(L.w13, D, 2 * L.ffp, 2);
+            else if (L.cfg.mlp.kind == FfnCfg::NONE) hint_next();
             const InMixerOutputs in{S.attn, S.mem, S.ssq, L.mem_norm, S.proj + L.proj.rg, L.md.H * L.md.vdim, L.md.vdim, L.md.nslice, eps};
             TRY((launch_gemv<WT, 1, false>(m, L.wo_l, S.attn, nullptr, nullptr, D, L.kl, EpiStore{S.y}, SrcPair{L.wo_r, D, L.kr, 0}, in)));
         }
         const FfnCfg& f = L.cfg.mlp;
         if (f.kind == FfnCfg::DENSE) {
             m->cur_cls = CLS_W13;
+            hint(L.w2, L.ffp, D, 1);
             TRY((launch_gemv<WT, 2, false>(m, L.w13, x[cur], nullptr, nullptr, 2 * L.ffp, D, EpiGate{S.gate, CD_ACT_SWIGLU}, SrcPlain{}, mix_in(L))));
             cur ^= 1;
             m->cur_cls = CLS_W2;
+            hint_next();
             TRY((launch_gemv<WT, 1, false>(m, L.w2, S.gate, nullptr, nullptr, D, L.ffp, EpiStore{S.y2})));
         } else if (f.kind == FfnCfg::MOE) {
             m->cur_cls = CLS_W13;
@@ -107,6 +120,7 @@ cudaError_t hybrid_step_t(cd_model* m, const cd_step& p) {
                 const SrcExpertRows s13{S.loc_ids, S.n_loc, nullptr, 2 * L.ffp, 0};
                 TRY((launch_gemv<WT, 2, false>(m, L.w13, x[cur], nullptr, nullptr, 2 * units, D, EpiGateMoe{S.gate, S.loc_w, S.n_loc, L.ffp}, s13)));
                 m->cur_cls = CLS_W2;
+                hint_next();
                 const SrcExpertCols s2{S.loc_ids, S.n_loc, nullptr, L.ffp, 0, D, (uint32_t)L.ffp * es, 0};
                 TRY((launch_gemv<WT, 1, false>(m, L.w2, S.gate, nullptr, nullptr, D, units, EpiStore{S.y2}, s2)));
             } else {
@@ -383,7 +397,10 @@ int build(const std::string& json, const SafeTensors* file, size_t max_tokens, c
         L.ad = AttnDims{a.heads, a.kv_heads, a.dim, a.vdim, pad_to(a.dim, 16), pad_to(a.vdim, 16), a.window, m->page_tokens, a.scale, h.eps, a.temp_coef, a.temp_every};
         L.md = MemDims{r.heads, r.dim, r.vdim, pad_to(r.vdim, 4), (r.vdim + MEM_SLICE - 1) / MEM_SLICE, r.gate_cap, h.eps};
         const size_t seen = a.window > 0 ? std::min<size_t>(a.window, max_tokens) : max_tokens;
-        L.nsplit = (int)std::max<size_t>(1, std::min<size_t>(32, (seen + MIX_TILE - 1) / MIX_TILE));
+        // slices of whole tiles, as many as one wave of CTAs has room for beside the memory's
+        const int tiles = (int)((seen + MIX_TILE - 1) / MIX_TILE), room = std::max(1, (4 * m->sm_count - L.md.H * L.md.nslice) / a.heads);
+        const int per_slice = std::max((tiles + 31) / 32, (tiles + room - 1) / room);
+        L.nsplit = std::max(1, (tiles + per_slice - 1) / per_slice);
         L.state_off = state;
         state += L.md.floats();
         mat(&L.wmix, pl.rows, D); mat(&L.wo_l, D, L.kl); mat(&L.wo_r, D, L.kr);

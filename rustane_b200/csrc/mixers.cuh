@@ -228,8 +228,25 @@ struct MixerStep {
     int nsplit;
 };
 constexpr int MIX_THREADS = 128, MIX_TILE = 32;
-__host__ __device__ inline size_t mixer_attn_smem_floats(int kp, int vp) { return (size_t)2 * kp + vp + (size_t)MIX_THREADS * 8 + MIX_TILE + 96; }
+__host__ __device__ inline size_t mixer_attn_smem_floats(int kp, int vp) { return (size_t)2 * kp + vp + (size_t)MIX_THREADS * 8 + 2 * MIX_TILE + 96; }
 __host__ __device__ inline size_t mixer_mem_smem_floats(int dim) { return (size_t)2 * dim + 4 * MEM_SLICE + 64; }
+
+// this thread's share of the sum of squares of n floats another kernel wrote
+__device__ inline float sum_of_squares(const float* v, int n) {
+    float s = 0.0f;
+    if ((n & 3) == 0 && (reinterpret_cast<size_t>(v) & 15) == 0) {
+        const float4* v4 = reinterpret_cast<const float4*>(v);
+#pragma unroll 8
+        for (int i = threadIdx.x; i < n / 4; i += MIX_THREADS) {
+            const float4 t = __ldcg(v4 + i);
+            s += t.x * t.x + t.y * t.y + t.z * t.z + t.w * t.w;
+        }
+    } else {
+#pragma unroll 8
+        for (int i = threadIdx.x; i < n; i += MIX_THREADS) { const float t = __ldcg(v + i); s = fmaf(t, t, s); }
+    }
+    return s;
+}
 
 // A matrix-memory slice: MEM_SLICE value columns of one head.  128 threads = 16 row groups x 8 column quads.
 __device__ inline void mem_step(const MixerStep& p, int idx, float* sm, float* red) {
@@ -326,6 +343,7 @@ __device__ inline void attn_step(const MixerStep& p, KT* __restrict__ pool, int 
     float* vc = kc + a.kp;                // [vp]
     float* accs = vc + a.vp;              // [128 threads][8]
     float* ps = accs + MIX_THREADS * 8;   // [MIX_TILE]
+    int* pages = reinterpret_cast<int*>(ps + MIX_TILE);  // [MIX_TILE] page of each position of the tile
     pdl_wait();
     pdl_launch_dependents();
     const int pos = __ldcg(&p.st->pos);
@@ -341,13 +359,9 @@ __device__ inline void attn_step(const MixerStep& p, KT* __restrict__ pool, int 
     while (lv < nvc) lv <<= 1;            // lanes that share a row of values
     const int vch = tid % lv, vgrp = tid / lv, vgroups = MIX_THREADS / lv;
     if (t0 < t1) {
-        float sq = 0.0f, sk = 0.0f;
         const bool newest = t1 == pos + 1;  // this slice holds the current position
-#pragma unroll 8
-        for (int i = tid; i < a.H * a.dim; i += MIX_THREADS) { const float v = __ldcg(p.proj + p.pl.lq + i); sq = fmaf(v, v, sq); }
-        if (newest)
-#pragma unroll 4
-            for (int i = tid; i < a.G * a.dim; i += MIX_THREADS) { const float v = __ldcg(p.proj + p.pl.lk + i); sk = fmaf(v, v, sk); }
+        if (tid < MIX_TILE) pages[tid] = p.page_table[min(t0 + tid, pos) / a.page_tokens];
+        const float sq = sum_of_squares(p.proj + p.pl.lq, a.H * a.dim), sk = newest ? sum_of_squares(p.proj + p.pl.lk, a.G * a.dim) : 0.0f;
         const float rq = a.temperature(pos) * a.scale / sqrtf(block_sum(sq, red) / (float)(a.H * a.dim) + a.eps);
         for (int i = tid; i < a.kp; i += MIX_THREADS)
             qs[i] = i < a.dim ? __ldcg(p.proj + p.pl.lq + h * a.dim + i) * rq * p.q_norm[h * a.dim + i] : 0.0f;
@@ -373,6 +387,16 @@ __device__ inline void attn_step(const MixerStep& p, KT* __restrict__ pool, int 
         const int kch = lane % lk, side = 32 / lk;
         const float slope = p.slopes[h];
         for (int tb = t0; tb < t1; tb += MIX_TILE) {
+            const int nt = min(MIX_TILE, t1 - tb);
+            // the tile's value rows are requested before its scores are worked out
+            constexpr int PRE = 4;
+            uint4 vw[PRE];
+#pragma unroll
+            for (int u = 0; u < PRE; ++u) {
+                const int j = vgrp + u * vgroups;
+                vw[u] = make_uint4(0, 0, 0, 0);
+                if (vch < nvc && j < nt && tb + j != pos) vw[u] = ldg_stream_coherent(pool + a.v_at(pages[j], g, (tb + j) % a.page_tokens) + (size_t)vch * EPC);
+            }
             // scores: warp w takes positions tb + 8 w .. + 7
             for (int j0 = 0; j0 < 8; j0 += 4 * side) {
                 float d[4] = {0.f, 0.f, 0.f, 0.f};
@@ -382,10 +406,7 @@ __device__ inline void attn_step(const MixerStep& p, KT* __restrict__ pool, int 
                     for (int u = 0; u < 4; ++u) {
                         const int j = j0 + u * side + lane / lk, t = tb + 8 * warp + j;
                         w[u] = make_uint4(0, 0, 0, 0);
-                        if (j < 8 && t < t1 && t != pos) {
-                            const int page = p.page_table[t / a.page_tokens];
-                            w[u] = ldg_stream_coherent(pool + a.k_at(page, g, t % a.page_tokens) + (size_t)c * EPC);
-                        }
+                        if (j < 8 && t < t1 && t != pos) w[u] = ldg_stream_coherent(pool + a.k_at(pages[8 * warp + j], g, t % a.page_tokens) + (size_t)c * EPC);
                     }
 #pragma unroll
                     for (int u = 0; u < 4; ++u) {
@@ -421,24 +442,29 @@ __device__ inline void attn_step(const MixerStep& p, KT* __restrict__ pool, int 
 #pragma unroll
             for (int e = 0; e < 8; ++e) acc[e] *= corr;
             if (vch < nvc) {
-                const int nt = min(MIX_TILE, t1 - tb);
-#pragma unroll 4
-                for (int j = vgrp; j < nt; j += vgroups) {
-                    const int tt = tb + j;
+                auto add = [&](int j, const uint4& raw) {
                     float f[EPC];
-                    if (tt == pos) {
+                    Elem<KT>::unpack(raw, f);
+                    if (tb + j == pos) {
 #pragma unroll
                         for (int e = 0; e < EPC; ++e) f[e] = vc[vch * EPC + e];
-                    } else {
-                        const int page = p.page_table[tt / a.page_tokens];
-                        Elem<KT>::unpack(ldg_stream_coherent(pool + a.v_at(page, g, tt % a.page_tokens) + (size_t)vch * EPC), f);
                     }
                     const float w = ps[j];
 #pragma unroll
                     for (int e = 0; e < EPC; ++e) acc[e] = fmaf(w, f[e], acc[e]);
-                }
+                };
+#pragma unroll
+                for (int u = 0; u < PRE; ++u)
+                    if (vgrp + u * vgroups < nt) add(vgrp + u * vgroups, vw[u]);
+#pragma unroll 4
+                for (int j = vgrp + PRE * vgroups; j < nt; j += vgroups)
+                    add(j, tb + j == pos ? make_uint4(0, 0, 0, 0) : ldg_stream_coherent(pool + a.v_at(pages[j], g, (tb + j) % a.page_tokens) + (size_t)vch * EPC));
             }
-            __syncthreads();
+            __syncthreads();  // the tile's pages and probabilities are no longer read
+            if (tb + MIX_TILE < t1) {
+                if (tid < MIX_TILE) pages[tid] = p.page_table[min(tb + MIX_TILE + tid, pos) / a.page_tokens];
+                __syncthreads();
+            }
         }
 #pragma unroll
         for (int e = 0; e < 8; ++e) accs[tid * 8 + e] = acc[e];
