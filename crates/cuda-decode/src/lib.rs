@@ -100,6 +100,11 @@ extern "C" {
                        opts: *const Options, out: *mut *mut c_void) -> c_int;
     fn cd_model_create_from_checkpoint(path: *const c_char, opts: *const Options, cfg_out: *mut Config,
                                        out: *mut *mut c_void) -> c_int;
+    fn cd_model_create_from_dir(dir: *const c_char, max_tokens: usize, opts: *const Options, out: *mut *mut c_void) -> c_int;
+    fn cd_model_get_config(m: *const c_void, cfg: *mut Config, opts: *mut Options, untied: *mut c_int) -> c_int;
+    fn cd_can_rewind(m: *const c_void, len: usize) -> c_int;
+    fn cd_prefill_logits(m: *mut c_void, ids: *const u32, n: usize, want: *const usize, nwant: usize, softcap: f32,
+                         out: *mut f32) -> c_int;
     fn cd_convert_checkpoint(src: *const c_char, dst: *const c_char, quant_dtype: c_int, device: c_int) -> c_int;
     fn cd_model_destroy(m: *mut c_void);
     fn cd_last_error(m: *const c_void) -> *const c_char;
@@ -184,6 +189,19 @@ impl Model {
         Ok(Self::wrap(out, cfg))
     }
 
+    /// A model folder (config.json, whose "architecture" the library's registry knows, and model.safetensors);
+    /// `max_tokens` (0: 4096) bounds the sequence.
+    pub fn from_dir(dir: &str, max_tokens: usize, opts: &Options) -> Result<Self, String> {
+        let c = CString::new(dir).map_err(|e| e.to_string())?;
+        let (mut cfg, mut out) = (Config::default(), std::ptr::null_mut());
+        let rc = unsafe { cd_model_create_from_dir(c.as_ptr(), max_tokens, opts, &mut out) };
+        if rc != 0 {
+            return Err(global_error());
+        }
+        unsafe { cd_model_get_config(out, &mut cfg, std::ptr::null_mut(), std::ptr::null_mut()) };
+        Ok(Self::wrap(out, cfg))
+    }
+
     /// Quantises the linears of an RSTK file once (`quant_dtype` 3: FP8-E4M3 with a scale per output row,
     /// 4: INT4 in groups of 32) and writes an RSTK v3 file that `from_checkpoint` streams into HBM as it is.
     pub fn convert_checkpoint(src: &str, dst: &str, quant_dtype: i32, device: i32) -> Result<(), String> {
@@ -229,6 +247,11 @@ impl Model {
     /// lib.rs:211-215 (clamped to seq)
     pub fn set_len(&mut self, len: usize) {
         self.check(unsafe { cd_set_len(self.h, len) })
+    }
+
+    /// Whether `set_len(len)` would succeed (families with recurrent state keep it at a few lengths only).
+    pub fn can_rewind(&self, len: usize) -> bool {
+        unsafe { cd_can_rewind(self.h, len) != 0 }
     }
 
     /// lib.rs:217-237: `k_rope_cf` and `v_cf` are channel-first `[kv_dim, seq]`.
@@ -319,6 +342,15 @@ impl Model {
     pub fn prefill(&mut self, ids: &[u32], softcap: f32, last_logits: Option<&mut [f32]>) -> Result<(), String> {
         let p = last_logits.map_or(std::ptr::null_mut(), |s| s.as_mut_ptr());
         self.fallible(unsafe { cd_prefill(self.h, ids.as_ptr(), ids.len(), softcap, p) })
+    }
+
+    /// The same with the logits after tokens `want` of this call, one row of `vocab` each.
+    pub fn prefill_logits(&mut self, ids: &[u32], want: &[usize], softcap: f32) -> Result<Vec<f32>, String> {
+        let mut out = vec![0f32; want.len() * self.cfg.vocab as usize];
+        self.fallible(unsafe {
+            cd_prefill_logits(self.h, ids.as_ptr(), ids.len(), want.as_ptr(), want.len(), softcap, out.as_mut_ptr())
+        })?;
+        Ok(out)
     }
 
     /// run_cached_sample's greedy loop (inference.rs:576-585) without a host round trip per token.

@@ -91,7 +91,7 @@ def weights(cfg, seed):
         elif name.endswith("f.b"):
             x = 2.5 + x
         elif leaf == "router":
-            x = 3.0 * x / np.sqrt(shape[1])
+            x = (3.0 if shape[0] < 32 else 12.0) * x / np.sqrt(shape[1])
         else:
             x = x / np.sqrt(shape[1])
         W[name] = bf16(x)
@@ -181,3 +181,7 @@ WIDE = config(256, 520, [                                 # head widths of real 
 ], eps=1e-5, mult=0.4)
 BROAD = config(128, 200, [(attn(2, 1, 192, 256, 48, 0.07), memory(1, 200, 264, 10.0), dense(128))], eps=1e-5, mult=1.0)
 LAST_MIXER = config(64, 130, [(attn(4, 2, 16, 16, 20, 0.3), memory(2, 16, 32, 8.0), None), (attn(1, 1, 32, 48, 9, 0.2), memory(4, 8, 12, 8.0), None)], mult=0.9)
+NARROW = config(72, 57, [                                 # widths that are no multiple of a GEMM chunk, many small experts
+    (attn(3, 3, 12, 4, 6, 0.6, 0.2, 2), memory(3, 6, 10, 7.0), moe(40, 6, 12, (10, 7))),
+    (attn(4, 1, 20, 28, 150, 0.25), memory(1, 4, 100, 7.0), dense(20)),
+], eps=1e-4, mult=0.6)

@@ -116,3 +116,21 @@ def test_short_prompts_and_fp32_models_keep_the_per_token_path(R, oracle):
     oc, om, gm = _models(R, oracle, (256, 640, 2, 128, 64, 2, 320), "bf16", {})
     cache, ref = _oracle_prefill(oracle, om, prompt[:5])
     assert float(np.abs(gm.prefill(prompt[:5]) - ref).max()) < 1e-3  # below the batching threshold
+
+
+@pytest.mark.parametrize("dtype", ["bf16", "f32"])
+def test_logits_at_chosen_places_of_a_prompt(R, oracle, dtype):
+    """cd_prefill_logits on the dense family, through the batched pass (bf16) and the per-token path (f32): the logits at
+    places in any order equal the oracle's, and a dense cache rewinds to any length."""
+    oc, om, gm = _models(R, oracle, (256, 640, 2, 128, 64, 2, 320), dtype, {})
+    prompt = oracle.synth_prompt(2, oc.vocab, 40)
+    cache = oracle.Cache(om, kv_round=0 if dtype == "f32" else 1)
+    ref = np.stack([cache.decode_logits(int(t)) for t in prompt])
+    want = [39, 0, 17, 17]
+    got = gm.prefill_logits(prompt, want)
+    assert float(np.abs(got - ref[want]).max()) < (1e-4 if dtype == "f32" else SPLIT_TOL)
+    assert gm.len() == 40 and gm.can_rewind(11)
+    gm.set_len(11)
+    assert float(np.abs(gm.prefill_logits(prompt[11:16], [4]) - ref[15]).max()) < (1e-4 if dtype == "f32" else SPLIT_TOL)
+    with pytest.raises(R.CudaDecodeError):
+        gm.prefill_logits(prompt[:3], [3])
