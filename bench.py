@@ -363,10 +363,9 @@ def bench_dafidra(sizes):
         sampler = ClockSampler(0)
         sampler.start()
         line["dafidra"] = measure(R.Model.from_config(cfg, 7, max_tokens=8192, use_graph=True), cfg["vocab"], dafidra_bytes(cfg, ctx), (1024, 2048, 4096))
-        if closest == "dense":
-            for label, mega in (("dense_per_operator", False), ("dense", True)):
-                line[label] = measure(R.Model.synthetic(R.Config(**dims), 7, dtype="bf16", use_graph=True, mega=mega), dims["vocab"], existing_bytes(closest, dims, ctx),
-                                      (1024, 2048, 4096))
+        if closest == "dense":  # (four query heads per kv head: one kernel per operator, like the configured decoder)
+            line[closest] = measure(R.Model.synthetic(R.Config(**dims), 7, dtype="bf16", use_graph=True), dims["vocab"], existing_bytes(closest, dims, ctx),
+                                    (1024, 2048, 4096))
         else:
             line[closest] = measure(R.Model.moe_synthetic(R.MoeConfig(**dims), 7, dtype="bf16", use_graph=True), dims["vocab"], existing_bytes(closest, dims, ctx), ())
         line["clocks"] = sampler.stop()

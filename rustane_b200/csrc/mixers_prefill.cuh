@@ -137,15 +137,14 @@ __global__ void __launch_bounds__(128) attn_window_kernel(const __grid_constant_
             uint32_t ah[4], al[4];
             ldsm_x4(ah, qh + a_off + (uint32_t)k * 32u);
             ldsm_x4(al, ql + a_off + (uint32_t)k * 32u);
+            uint32_t b[4][4];
 #pragma unroll
-            for (int n = 0; n < 4; ++n) {
-                uint32_t b[4];
-                ldsm_x4(b, kt + b_off + (uint32_t)(16 * n) * ldk + (uint32_t)k * 32u);
-                Mma16<KT>::mma(s[2 * n], ah, b[0], b[1]);
-                Mma16<KT>::mma(s[2 * n], al, b[0], b[1]);
-                Mma16<KT>::mma(s[2 * n + 1], ah, b[2], b[3]);
-                Mma16<KT>::mma(s[2 * n + 1], al, b[2], b[3]);
-            }
+            for (int n = 0; n < 4; ++n) ldsm_x4(b[n], kt + b_off + (uint32_t)(16 * n) * ldk + (uint32_t)k * 32u);
+            // the two products of an accumulator are kept apart: back to back the second would wait for the first
+#pragma unroll
+            for (int n = 0; n < 4; ++n) { Mma16<KT>::mma(s[2 * n], ah, b[n][0], b[n][1]); Mma16<KT>::mma(s[2 * n + 1], ah, b[n][2], b[n][3]); }
+#pragma unroll
+            for (int n = 0; n < 4; ++n) { Mma16<KT>::mma(s[2 * n], al, b[n][0], b[n][1]); Mma16<KT>::mma(s[2 * n + 1], al, b[n][2], b[n][3]); }
         }
         const int j0 = lo + tile * AW_TILE + 2 * tq;
         float x_a = NEG, x_b = NEG;
@@ -187,14 +186,21 @@ __global__ void __launch_bounds__(128) attn_window_kernel(const __grid_constant_
             const uint32_t pl[4] = {pack2<KT>(s0[0] - round16<KT>(s0[0]), s0[1] - round16<KT>(s0[1])), pack2<KT>(s0[2] - round16<KT>(s0[2]), s0[3] - round16<KT>(s0[3])),
                                     pack2<KT>(s1[0] - round16<KT>(s1[0]), s1[1] - round16<KT>(s1[1])), pack2<KT>(s1[2] - round16<KT>(s1[2]), s1[3] - round16<KT>(s1[3]))};
 #pragma unroll
-            for (int n = 0; n < VD / 16; ++n) {
+            for (int n = 0; n < VD / 16; n += 2) {
                 if (16 * n < a.vp) {
-                    uint32_t b[4];
+                    const bool two = 16 * (n + 1) < a.vp;
+                    uint32_t b[4], c[4];
                     ldsm_x4_trans(b, vt + v_off + (uint32_t)(16 * k) * ldv + (uint32_t)n * 32u);
+                    if (two) ldsm_x4_trans(c, vt + v_off + (uint32_t)(16 * k) * ldv + (uint32_t)(n + 1) * 32u);
+                    else c[0] = c[1] = c[2] = c[3] = 0u;
                     Mma16<KT>::mma(o[2 * n], ph, b[0], b[1]);
-                    Mma16<KT>::mma(o[2 * n], pl, b[0], b[1]);
                     Mma16<KT>::mma(o[2 * n + 1], ph, b[2], b[3]);
+                    Mma16<KT>::mma(o[2 * n + 2], ph, c[0], c[1]);
+                    Mma16<KT>::mma(o[2 * n + 3], ph, c[2], c[3]);
+                    Mma16<KT>::mma(o[2 * n], pl, b[0], b[1]);
                     Mma16<KT>::mma(o[2 * n + 1], pl, b[2], b[3]);
+                    Mma16<KT>::mma(o[2 * n + 2], pl, c[0], c[1]);
+                    Mma16<KT>::mma(o[2 * n + 3], pl, c[2], c[3]);
                 }
             }
         }
@@ -276,6 +282,7 @@ __device__ inline void mem_chunk_gates(const MemPrompt& p, int h, int t0, int nt
 
 // a [64][64] tile of fp32 rows as bf16 head and remainder; rows >= nrows and columns >= ncols are zero; row_scale may be null
 __device__ inline void mem_load_tile(__nv_bfloat16* hi, __nv_bfloat16* lo, const float* src, size_t ld, int nrows, int ncols, const float* row_scale, float scale) {
+#pragma unroll 8
     for (int i = threadIdx.x; i < 64 * 64; i += 128) {
         const int r = i >> 6, c = i & 63;
         float v = 0.0f;
@@ -284,6 +291,17 @@ __device__ inline void mem_load_tile(__nv_bfloat16* hi, __nv_bfloat16* lo, const
     }
 }
 constexpr int MEM_TILE_ELEMS = 64 * MEM_LD;
+
+// the three products of every accumulator, kept apart (back to back each would wait for the one before)
+__device__ inline void mem_mma3(float (&acc)[8][4], const uint32_t (&ah)[4], const uint32_t (&al)[4], const uint32_t (&bh)[4][4], const uint32_t (&bl)[4][4]) {
+    typedef Mma16<__nv_bfloat16> X;
+#pragma unroll
+    for (int n = 0; n < 4; ++n) { X::mma(acc[2 * n], ah, bh[n][0], bh[n][1]); X::mma(acc[2 * n + 1], ah, bh[n][2], bh[n][3]); }
+#pragma unroll
+    for (int n = 0; n < 4; ++n) { X::mma(acc[2 * n], ah, bl[n][0], bl[n][1]); X::mma(acc[2 * n + 1], ah, bl[n][2], bl[n][3]); }
+#pragma unroll
+    for (int n = 0; n < 4; ++n) { X::mma(acc[2 * n], al, bh[n][0], bh[n][1]); X::mma(acc[2 * n + 1], al, bh[n][2], bh[n][3]); }
+}
 
 // acc[64 columns] of this warp's 16 rows += A B with three products of the heads and remainders; A fragments from
 // `load_a(k, hi, lo)`, B stored [k][64] in (bhi, blo)
@@ -295,18 +313,13 @@ __device__ inline void mem_mma_kn(float (&acc)[8][4], uint32_t bhi, uint32_t blo
     for (int k = 0; k < 4; ++k) {
         uint32_t ah[4], al[4];
         load_a(k, ah, al);
+        uint32_t bh[4][4], bl[4][4];
 #pragma unroll
         for (int n = 0; n < 4; ++n) {
-            uint32_t bh[4], bl[4];
-            ldsm_x4_trans(bh, bhi + off + (uint32_t)(16 * k) * (MEM_LD * 2) + (uint32_t)n * 32u);
-            ldsm_x4_trans(bl, blo + off + (uint32_t)(16 * k) * (MEM_LD * 2) + (uint32_t)n * 32u);
-            Mma16<__nv_bfloat16>::mma(acc[2 * n], ah, bh[0], bh[1]);
-            Mma16<__nv_bfloat16>::mma(acc[2 * n], ah, bl[0], bl[1]);
-            Mma16<__nv_bfloat16>::mma(acc[2 * n], al, bh[0], bh[1]);
-            Mma16<__nv_bfloat16>::mma(acc[2 * n + 1], ah, bh[2], bh[3]);
-            Mma16<__nv_bfloat16>::mma(acc[2 * n + 1], ah, bl[2], bl[3]);
-            Mma16<__nv_bfloat16>::mma(acc[2 * n + 1], al, bh[2], bh[3]);
+            ldsm_x4_trans(bh[n], bhi + off + (uint32_t)(16 * k) * (MEM_LD * 2) + (uint32_t)n * 32u);
+            ldsm_x4_trans(bl[n], blo + off + (uint32_t)(16 * k) * (MEM_LD * 2) + (uint32_t)n * 32u);
         }
+        mem_mma3(acc, ah, al, bh, bl);
     }
 }
 
@@ -463,18 +476,13 @@ static __global__ void __launch_bounds__(128) mem_out_kernel(const __grid_consta
             uint32_t ah[4], al[4];
             ldsm_x4(ah, qha + a_off + (uint32_t)k * 32u);
             ldsm_x4(al, qla + a_off + (uint32_t)k * 32u);
+            uint32_t bh[4][4], bl[4][4];
 #pragma unroll
             for (int n = 0; n < 4; ++n) {
-                uint32_t bh[4], bl[4];
-                ldsm_x4(bh, kha + b_off + (uint32_t)(16 * n) * (MEM_LD * 2) + (uint32_t)k * 32u);
-                ldsm_x4(bl, kla + b_off + (uint32_t)(16 * n) * (MEM_LD * 2) + (uint32_t)k * 32u);
-                Mma16<__nv_bfloat16>::mma(sc[2 * n], ah, bh[0], bh[1]);
-                Mma16<__nv_bfloat16>::mma(sc[2 * n], ah, bl[0], bl[1]);
-                Mma16<__nv_bfloat16>::mma(sc[2 * n], al, bh[0], bh[1]);
-                Mma16<__nv_bfloat16>::mma(sc[2 * n + 1], ah, bh[2], bh[3]);
-                Mma16<__nv_bfloat16>::mma(sc[2 * n + 1], ah, bl[2], bl[3]);
-                Mma16<__nv_bfloat16>::mma(sc[2 * n + 1], al, bh[2], bh[3]);
+                ldsm_x4(bh[n], kha + b_off + (uint32_t)(16 * n) * (MEM_LD * 2) + (uint32_t)k * 32u);
+                ldsm_x4(bl[n], kla + b_off + (uint32_t)(16 * n) * (MEM_LD * 2) + (uint32_t)k * 32u);
             }
+            mem_mma3(sc, ah, al, bh, bl);
         }
         mem_mma_kn(o, smem_addr(sh), smem_addr(sl), [&](int k, uint32_t (&ah)[4], uint32_t (&al)[4]) {
             ldsm_x4(ah, qha + a_off + (uint32_t)k * 32u);
