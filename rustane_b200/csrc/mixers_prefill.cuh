@@ -1,5 +1,5 @@
 // The configured decoder's mixers, routing and vector steps over many prompt tokens at once (tensor cores: mma.sync for
-// the two mixers, whose operands are produced in the kernel; the linears are pf_gemm_kernel, prefill.cuh).  Same
+// the mixers, whose operands are produced in the kernel; the linears are pf_gemm_kernel, prefill.cuh).  Same
 // arithmetic as the one-token kernels of mixers.cuh; fp32 operands enter the tensor cores as a 16-bit value and a 16-bit
 // remainder, so a product keeps 16 (bf16) or 22 (fp16) mantissa bits.
 #pragma once
@@ -19,29 +19,48 @@ template <typename T> __device__ inline uint32_t pack2(float a, float b) {
 template <typename T> __device__ inline float round16(float v) { return Elem<T>::to_f32(Elem<T>::from_f32(v)); }
 
 // ---------------------------------------------------------------------- after the projections: q, k and v of the attention
-// One CTA per token: whole-projection norms, temperature on q; q as 16-bit head and remainder [rows][H * kp], the key and
-// value rows into their pages.
+// One CTA per token: whole-projection norms or rotation, temperature on q; q as 16-bit head and remainder
+// [rows][H * maps * kp], the key and value rows into their pages.
 template <typename KT>
 __global__ void __launch_bounds__(256) attn_rows_kernel(const float* __restrict__ proj, int ld, AttnDims a, ProjLayout pl, const float* __restrict__ q_norm,
                                                         const float* __restrict__ k_norm, const int* __restrict__ page_table, KT* __restrict__ pool,
                                                         KT* __restrict__ q_hi, KT* __restrict__ q_lo, int pos0) {
     __shared__ float red[32];
     const float* row = proj + (size_t)blockIdx.x * ld;
-    const int pos = pos0 + blockIdx.x, tid = threadIdx.x;
-    float sq = 0.0f, sk = 0.0f;
-    for (int i = tid; i < a.H * a.dim; i += 256) sq = fmaf(row[pl.lq + i], row[pl.lq + i], sq);
-    for (int i = tid; i < a.G * a.dim; i += 256) sk = fmaf(row[pl.lk + i], row[pl.lk + i], sk);
-    const float rq = a.temperature(pos) / sqrtf(block_sum(sq, red) / (float)(a.H * a.dim) + a.eps);
-    const float rk = 1.0f / sqrtf(block_sum(sk, red) / (float)(a.G * a.dim) + a.eps);
-    for (int i = tid; i < a.H * a.kp; i += 256) {
-        const int h = i / a.kp, d = i % a.kp;
-        const float v = d < a.dim ? row[pl.lq + h * a.dim + d] * rq * q_norm[h * a.dim + d] : 0.0f;
-        pf_store(q_hi, q_lo, (size_t)blockIdx.x * a.H * a.kp + i, v);
+    const int pos = pos0 + blockIdx.x, tid = threadIdx.x, nq = a.H * a.maps * a.dim, nk = a.G * a.maps * a.dim;
+    float rq = a.temperature(pos), rk = 1.0f;
+    if (q_norm != nullptr) {
+        float sq = 0.0f, sk = 0.0f;
+        for (int i = tid; i < nq; i += 256) sq = fmaf(row[pl.lq + i], row[pl.lq + i], sq);
+        for (int i = tid; i < nk; i += 256) sk = fmaf(row[pl.lk + i], row[pl.lk + i], sk);
+        rq /= sqrtf(block_sum(sq, red) / (float)nq + a.eps);
+        rk = 1.0f / sqrtf(block_sum(sk, red) / (float)nk + a.eps);
+    }
+    // two neighbouring entries (a rotated pair) of a [head][map][kp] vector
+    auto pair = [&](const float* src, const float* norm, int i, float r, float& u, float& v) {
+        const int hm = i / a.kp, d = i % a.kp;
+        const float* p = src + hm * a.dim;
+        u = d < a.dim ? p[d] * r * (norm != nullptr ? norm[hm * a.dim + d] : 1.0f) : 0.0f;
+        v = d + 1 < a.dim ? p[d + 1] * r * (norm != nullptr ? norm[hm * a.dim + d + 1] : 1.0f) : 0.0f;
+        if (d < a.rot.dims) {
+            const float2 cs = a.rot.at(pos, d >> 1);
+            const float t = u * cs.x - v * cs.y;
+            v = v * cs.x + u * cs.y;
+            u = t;
+        }
+    };
+    float u, v;
+    for (int i = 2 * tid; i < a.H * a.kr(); i += 512) {
+        pair(row + pl.lq, q_norm, i, rq, u, v);
+        pf_store(q_hi, q_lo, (size_t)blockIdx.x * a.H * a.kr() + i, u);
+        pf_store(q_hi, q_lo, (size_t)blockIdx.x * a.H * a.kr() + i + 1, v);
     }
     const int page = page_table[pos / a.page_tokens], off = pos % a.page_tokens;
-    for (int i = tid; i < a.G * a.kp; i += 256) {
-        const int g = i / a.kp, d = i % a.kp;
-        pool[a.k_at(page, g, off) + d] = Elem<KT>::from_f32(d < a.dim ? row[pl.lk + g * a.dim + d] * rk * k_norm[g * a.dim + d] : 0.0f);
+    for (int i = 2 * tid; i < a.G * a.kr(); i += 512) {
+        pair(row + pl.lk, k_norm, i, rk, u, v);
+        KT* k = pool + a.k_at(page, i / a.kr(), off) + i % a.kr();
+        k[0] = Elem<KT>::from_f32(u);
+        k[1] = Elem<KT>::from_f32(v);
     }
     for (int i = tid; i < a.G * a.vp; i += 256) {
         const int g = i / a.vp, d = i % a.vp;
@@ -50,7 +69,7 @@ __global__ void __launch_bounds__(256) attn_rows_kernel(const float* __restrict_
 }
 
 // ---------------------------------------------------------------------- windowed attention of the prompt
-// grid = (ceil(rows / 64), heads), four warps of 16 query rows.  Keys of the window are walked 64 at a time straight out
+// grid = (ceil(rows / 64), heads * maps), four warps of 16 query rows.  Visible keys are walked 64 at a time straight out
 // of the pages (cp.async, two tiles in flight), scores and the running softmax stay in registers.
 constexpr int AW_TILE = 64;
 __host__ __device__ inline size_t attn_window_smem(int kp, int vp) { return (size_t)AW_TILE * (4 * (kp + 8) + 2 * (vp + 8)) * 2; }
@@ -63,13 +82,14 @@ template <int N> __device__ inline void cp_async_wait() { asm volatile("cp.async
 
 struct AttnWindow {
     AttnDims a;
-    const float* slopes;
-    const float* sink;
-    const float* proj;     // gate projections: row ld, column gate_off + head
+    const float* slopes;   // nullptr: no distance bias
+    const float* sink;     // nullptr: none
+    const float* proj;     // gate projections: row ld, column gate_off + head (a gate per head is applied here)
     int proj_ld, gate_off;
     const int* page_table;
     int rows, pos0;        // query rows and the position of the first
-    int out_ld;            // row stride of the gated output [rows][H * vdim], padded with zeros
+    int out_ld;            // row stride of the output [rows][H * vdim], padded with zeros
+    float* raw;            // not nullptr: the maps' outputs [rows][H * maps][vdim] go here instead, in fp32
 };
 
 template <typename KT, typename AT, int VD>
@@ -78,8 +98,8 @@ __global__ void __launch_bounds__(128) attn_window_kernel(const __grid_constant_
     extern __shared__ __align__(128) unsigned char aw_raw[];
     constexpr float NEG = -3.402823466e+38f;
     const AttnDims& a = p.a;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h = blockIdx.y, g = h / (a.H / a.G);
-    const int r0 = blockIdx.x * AW_TILE;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, hm = blockIdx.y, h = hm / a.maps, g = h / (a.H / a.G);
+    const int r0 = blockIdx.x * AW_TILE, map_off = (hm % a.maps) * a.kp;
     const uint32_t ldk = (uint32_t)(a.kp + 8) * 2u, ldv = (uint32_t)(a.vp + 8) * 2u;
     const uint32_t qh = smem_addr(aw_raw), ql = qh + AW_TILE * ldk, ks0 = ql + AW_TILE * ldk, vs0 = ks0 + 2 * AW_TILE * ldk;
     const int p_first = p.pos0 + r0, p_last = min(p.pos0 + p.rows, p.pos0 + r0 + AW_TILE) - 1;
@@ -89,7 +109,7 @@ __global__ void __launch_bounds__(128) attn_window_kernel(const __grid_constant_
     for (int i = tid; i < AW_TILE * kch; i += 128) {
         const int r = i / kch, c = i % kch;
         const bool ok = r0 + r < p.rows;
-        const size_t at = ((size_t)(ok ? r0 + r : 0) * a.H + h) * a.kp + c * 8;
+        const size_t at = ((size_t)(ok ? r0 + r : 0) * a.H * a.maps + hm) * a.kp + c * 8;
         cp_async16(qh + r * ldk + c * 16, q_hi + at, ok ? 16 : 0);
         cp_async16(ql + r * ldk + c * 16, q_lo + at, ok ? 16 : 0);
     }
@@ -99,7 +119,7 @@ __global__ void __launch_bounds__(128) attn_window_kernel(const __grid_constant_
             const int r = i / kch, c = i % kch, t = lo + tile * AW_TILE + r;
             const bool ok = t <= p_last;
             const int tt = ok ? t : p_last;
-            cp_async16(kd + r * ldk + c * 16, pool + a.k_at(p.page_table[tt / a.page_tokens], g, tt % a.page_tokens) + c * 8, ok ? 16 : 0);
+            cp_async16(kd + r * ldk + c * 16, pool + a.k_at(p.page_table[tt / a.page_tokens], g, tt % a.page_tokens) + map_off + c * 8, ok ? 16 : 0);
         }
         for (int i = tid; i < AW_TILE * vch; i += 128) {
             const int r = i / vch, c = i % vch, t = lo + tile * AW_TILE + r;
@@ -113,7 +133,7 @@ __global__ void __launch_bounds__(128) attn_window_kernel(const __grid_constant_
     const int gq = lane >> 2, tq = lane & 3;
     const int row_a = r0 + 16 * warp + gq, row_b = row_a + 8;  // this lane's two query rows
     const int pa = p.pos0 + row_a, pb = p.pos0 + row_b;
-    const float slope = p.slopes[h];
+    const float slope = p.slopes != nullptr ? p.slopes[h] : 0.0f;
     float m_a = NEG, m_b = NEG, l_a = 0.0f, l_b = 0.0f;
     float o[VD / 8][4];
 #pragma unroll
@@ -211,11 +231,12 @@ __global__ void __launch_bounds__(128) attn_window_kernel(const __grid_constant_
         l_a += __shfl_xor_sync(0xffffffffu, l_a, w);
         l_b += __shfl_xor_sync(0xffffffffu, l_b, w);
     }
-    const float sink = p.sink[h];
+    const float sink = p.sink != nullptr ? p.sink[h] : NEG;
     auto finish = [&](int row, float m, float l) {  // factor of the row's accumulators: sink in the denominator, head gate
         if (row >= p.rows) return 0.0f;
         const float M = fmaxf(m, sink), e = expf(m - M);
-        return e / (l * e + expf(sink - M)) * sigmoid(p.proj[(size_t)row * p.proj_ld + p.gate_off + h]);
+        const float f = e / (l * e + (p.sink != nullptr ? expf(sink - M) : 0.0f));
+        return a.gate == 1 ? f * sigmoid(p.proj[(size_t)row * p.proj_ld + p.gate_off + h]) : f;
     };
     const float f_a = finish(row_a, m_a, l_a), f_b = finish(row_b, m_b, l_b);
 #pragma unroll
@@ -224,15 +245,129 @@ __global__ void __launch_bounds__(128) attn_window_kernel(const __grid_constant_
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
             if (c + e < a.vdim) {
-                if (row_a < p.rows) pf_store(out_hi, out_lo, (size_t)row_a * p.out_ld + h * a.vdim + c + e, o[n][e] * f_a);
-                if (row_b < p.rows) pf_store(out_hi, out_lo, (size_t)row_b * p.out_ld + h * a.vdim + c + e, o[n][2 + e] * f_b);
+                if (p.raw != nullptr) {
+                    if (row_a < p.rows) p.raw[((size_t)row_a * a.H * a.maps + hm) * a.vdim + c + e] = o[n][e] * f_a;
+                    if (row_b < p.rows) p.raw[((size_t)row_b * a.H * a.maps + hm) * a.vdim + c + e] = o[n][2 + e] * f_b;
+                } else {
+                    if (row_a < p.rows) pf_store(out_hi, out_lo, (size_t)row_a * p.out_ld + h * a.vdim + c + e, o[n][e] * f_a);
+                    if (row_b < p.rows) pf_store(out_hi, out_lo, (size_t)row_b * p.out_ld + h * a.vdim + c + e, o[n][2 + e] * f_b);
+                }
             }
         }
     }
+    if (p.raw != nullptr) return;
     if (h == a.H - 1)
         for (int r = tid; r < AW_TILE && r0 + r < p.rows; r += 128)
             for (int c = a.H * a.vdim; c < p.out_ld; ++c) pf_store(out_hi, out_lo, (size_t)(r0 + r) * p.out_ld + c, 0.0f);
 }
+
+// per token: the second map's output subtracted from the first's, each head divided by its root mean square, times the
+// constant factor and the gate of every element; one warp per head
+template <typename AT>
+__global__ void __launch_bounds__(256) diff_rows_kernel(const float* __restrict__ raw, const float* __restrict__ proj, int proj_ld, int gate_off, AttnDims a,
+                                                        AT* __restrict__ hi, AT* __restrict__ lo, int ld) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const float* gate = proj + (size_t)blockIdx.x * proj_ld + gate_off;
+    for (int h = warp; h < a.H; h += 8) {
+        const float* o1 = raw + ((size_t)blockIdx.x * a.H + h) * 2 * a.vdim;
+        const float* o2 = o1 + a.vdim;
+        float ss = 0.0f;
+        for (int i = lane; i < a.vdim; i += 32) { const float v = o1[i] - a.lambda * o2[i]; ss = fmaf(v, v, ss); }
+        const float r = a.out_scale / sqrtf(warp_sum(ss) / (float)a.vdim + a.eps);
+        for (int i = lane; i < a.vdim; i += 32) {
+            const int j = h * a.vdim + i;
+            pf_store(hi, lo, (size_t)blockIdx.x * ld + j, (o1[i] - a.lambda * o2[i]) * r * (a.gate == 2 ? sigmoid(gate[j]) : a.gate == 1 ? sigmoid(gate[h]) : 1.0f));
+        }
+    }
+    for (int j = a.H * a.vdim + threadIdx.x; j < ld; j += 256) pf_store(hi, lo, (size_t)blockIdx.x * ld + j, 0.0f);
+}
+
+// ---------------------------------------------------------------------- latent attention of the prompt
+// Keys and values of the visible positions are expanded once per piece into a buffer laid out like one page, then attended
+// to by attn_window_kernel.  latent_rows_kernel: one CTA per new token, q as 16-bit head and remainder [rows][H][kp], the
+// cache row [normed latent | rotated key].
+template <typename KT>
+__global__ void __launch_bounds__(256) latent_rows_kernel(const float* __restrict__ proj, int ld, MlaDims d, Rotation rot, const float* __restrict__ gamma,
+                                                          const int* __restrict__ page_table, KT* __restrict__ pool, KT* __restrict__ q_hi, KT* __restrict__ q_lo,
+                                                          int kp, int pos0) {
+    __shared__ float red[32];
+    const float* row = proj + (size_t)blockIdx.x * ld;
+    const int pos = pos0 + blockIdx.x, tid = threadIdx.x, QH = d.nope_n + d.rope_n;
+    for (int i = tid; i < d.heads * kp; i += 256) {
+        const int h = i / kp, k = i % kp;
+        const float* q = row + h * QH;
+        const float v = k < d.nope_n ? q[k] : k < QH ? rot.entry(pos, k - d.nope_n, [&](int j) { return q[d.nope_n + j]; }) : 0.0f;
+        pf_store(q_hi, q_lo, (size_t)blockIdx.x * d.heads * kp + i, v);
+    }
+    const float* craw = row + d.heads * QH;
+    float ss = 0.0f;
+    for (int i = tid; i < d.latent_n; i += 256) ss = fmaf(craw[i], craw[i], ss);
+    const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)d.latent_n + d.eps);
+    KT* out = pool + ((size_t)page_table[pos / d.page_tokens] * d.page_tokens + pos % d.page_tokens) * d.row();
+    for (int i = tid; i < d.latent; i += 256) out[i] = Elem<KT>::from_f32(i < d.latent_n ? craw[i] * r * gamma[i] : 0.0f);
+    for (int i = tid; i < d.rope; i += 256) out[d.latent + i] = Elem<KT>::from_f32(i < d.rope_n ? rot.entry(pos, i, [&](int j) { return craw[d.latent_n + j]; }) : 0.0f);
+}
+
+// cached rows base, base + 1, ..: the latent as a GEMM operand [n][latent], the rotated key behind every head's expanded one
+// (`x` describes the expanded buffer), zeros in its padding.  One CTA per position.
+template <typename KT, typename AT>
+__global__ void __launch_bounds__(256) latent_gather_kernel(const KT* __restrict__ pool, const int* __restrict__ page_table, MlaDims d, int base, AT* __restrict__ hi,
+                                                            AT* __restrict__ lo, KT* __restrict__ expanded, AttnDims x) {
+    const int pos = base + blockIdx.x, tid = threadIdx.x;
+    const KT* row = pool + ((size_t)page_table[pos / d.page_tokens] * d.page_tokens + pos % d.page_tokens) * d.row();
+    for (int i = tid; i < d.latent; i += 256) pf_store(hi, lo, (size_t)blockIdx.x * d.latent + i, Elem<KT>::to_f32(row[i]));
+    const int nk = x.kp - d.nope_n, nv = x.vp - x.vdim;
+    const KT zero = Elem<KT>::from_f32(0.0f);
+    for (int i = tid; i < x.H * nk; i += 256) {
+        const int h = i / nk, k = i % nk;
+        expanded[x.k_at(0, h, blockIdx.x) + d.nope_n + k] = k < d.rope_n ? row[d.latent + k] : zero;
+    }
+    for (int i = tid; i < x.H * nv; i += 256) expanded[x.v_at(0, i / nv, blockIdx.x) + x.vdim + i % nv] = zero;
+}
+
+// output columns [H][nope] keys, then [H][vdim] values, of the expansion GEMM
+template <typename KT> struct PfEpiExpand {
+    KT* expanded;
+    AttnDims x;
+    int nope;
+    __device__ void operator()(int, int row, int col, const float (&v)[32]) const {
+        const int keys = x.H * nope;
+        int h = col < keys ? col / nope : (col - keys) / x.vdim, d = col < keys ? col % nope : (col - keys) % x.vdim;
+        bool key = col < keys;
+        if (h >= x.H) return;
+        KT* dst = expanded + (key ? x.k_at(0, h, row) : x.v_at(0, h, row));
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+            dst[d] = Elem<KT>::from_f32(v[i]);
+            if (++d == (key ? nope : x.vdim)) {
+                d = 0;
+                if (++h == x.H) {
+                    if (!key) return;  // columns past the last value
+                    key = false;
+                    h = 0;
+                }
+                dst = expanded + (key ? x.k_at(0, h, row) : x.v_at(0, h, row));
+            }
+        }
+    }
+};
+
+// ---------------------------------------------------------------------- token side: gate of the second embedding's part
+template <typename AT, typename WT> struct PfEpiTokenGate {
+    AT *hi, *lo;
+    int ld;               // columns of the operand, zeros behind `dim`
+    const WT* table;      // the layer's first column
+    int table_ld, dim;
+    const uint32_t* ids;
+    __device__ void operator()(int, int row, int col, const float (&v)[32]) const {
+        const WT* e = table + (size_t)ids[row] * table_ld;
+#pragma unroll
+        for (int i = 0; i < 32; ++i) {
+            const int c = col + i;
+            if (c < ld) pf_store(hi, lo, (size_t)row * ld + c, c < dim ? gelu_tanh(v[i]) * Elem<WT>::to_f32(e[c]) : 0.0f);
+        }
+    }
+};
 
 // ---------------------------------------------------------------------- matrix memory of the prompt, chunk by chunk
 // With F_t the running sum of the log forget gates inside a chunk and a_s = i_s - F_s, the recurrence unrolls to
@@ -240,6 +375,8 @@ __global__ void __launch_bounds__(128) attn_window_kernel(const __grid_constant_
 //   S_t^T q = e^{m_0 - M_t} S_0^T q + sum_{s <= t} e^{a_s - M_t} (k_s . q) v_s     (n . q likewise),
 // so a chunk needs only the state it starts from.  Three kernels: every chunk's own contribution to the state, a scan over
 // the chunks that turns the contributions into starting states, and the read-outs of all chunks.
+// Linear attention is the case with log forget gate ln(decay), input gate 1 and no maximum or normaliser: F_t = (t + 1) ln
+// decay, every scale e^0, and M_t = -F_t in the read-out.
 struct MemPrompt {
     MemDims d;
     ProjLayout pl;
@@ -259,6 +396,14 @@ struct MemPrompt {
 // end forget nothing and add nothing.  Ends with a barrier.
 __device__ inline void mem_chunk_gates(const MemPrompt& p, int h, int t0, int nt, float* F, float* I, float* tmp) {
     const int tid = threadIdx.x;
+    if (p.d.linear()) {
+        if (tid < MEM_CHUNK) {
+            F[tid] = (float)min(tid + 1, nt) * p.d.log_decay[h];
+            I[tid] = tid < nt ? 0.0f : -INFINITY;
+        }
+        __syncthreads();
+        return;
+    }
     if (tid < MEM_CHUNK) {
         float gi = -INFINITY, gf = 0.0f;
         if (tid < nt) {
@@ -280,13 +425,16 @@ __device__ inline void mem_chunk_gates(const MemPrompt& p, int h, int t0, int nt
     __syncthreads();
 }
 
-// a [64][64] tile of fp32 rows as bf16 head and remainder; rows >= nrows and columns >= ncols are zero; row_scale may be null
-__device__ inline void mem_load_tile(__nv_bfloat16* hi, __nv_bfloat16* lo, const float* src, size_t ld, int nrows, int ncols, const float* row_scale, float scale) {
+// a [64][64] tile of fp32 rows (act: through silu) as bf16 head and remainder; rows >= nrows and columns >= ncols are zero; row_scale may be null
+__device__ inline void mem_load_tile(__nv_bfloat16* hi, __nv_bfloat16* lo, const float* src, size_t ld, int nrows, int ncols, const float* row_scale, float scale, bool act = false) {
 #pragma unroll 8
     for (int i = threadIdx.x; i < 64 * 64; i += 128) {
         const int r = i >> 6, c = i & 63;
         float v = 0.0f;
-        if (r < nrows && c < ncols) v = src[(size_t)r * ld + c] * (row_scale ? row_scale[r] : scale);
+        if (r < nrows && c < ncols) {
+            v = src[(size_t)r * ld + c];
+            v = (act ? silu(v) : v) * (row_scale ? row_scale[r] : scale);
+        }
         pf_store(hi, lo, (size_t)r * MEM_LD + c, v);
     }
 }
@@ -332,14 +480,15 @@ static __global__ void __launch_bounds__(128) mem_chunk_kernel(const __grid_cons
     const int t0 = c * MEM_CHUNK, nt = min(MEM_CHUNK, p.rows - t0);
     mem_chunk_gates(p, h, t0, nt, F, I, &tmp);
     const float Fend = F[MEM_CHUNK - 1];
-    float wmax = -INFINITY;
-    for (int s = 0; s < nt; ++s) wmax = fmaxf(wmax, Fend - F[s] + I[s]);
+    const bool linear = d.linear();
+    float wmax = linear ? 0.0f : -INFINITY;
+    for (int s = 0; s < nt && !linear; ++s) wmax = fmaxf(wmax, Fend - F[s] + I[s]);
     if (tid < MEM_CHUNK) W[tid] = expf(Fend - F[tid] + I[tid] - wmax);
     __syncthreads();
     __nv_bfloat16 *kh = tiles, *kl = tiles + MEM_TILE_ELEMS, *vh = tiles + 2 * MEM_TILE_ELEMS, *vl = tiles + 3 * MEM_TILE_ELEMS;
     const float* row0 = p.proj + (size_t)t0 * p.proj_ld;
-    mem_load_tile(kh, kl, row0 + p.pl.rk + h * d.dim + kb * 64, p.proj_ld, nt, d.dim - kb * 64, W, 1.0f);
-    mem_load_tile(vh, vl, row0 + p.pl.rv + h * d.vdim + vb * 64, p.proj_ld, nt, d.vdim - vb * 64, nullptr, 1.0f);
+    mem_load_tile(kh, kl, row0 + p.pl.rk + h * d.dim + kb * 64, p.proj_ld, nt, d.dim - kb * 64, W, 1.0f, linear);
+    mem_load_tile(vh, vl, row0 + p.pl.rv + h * d.vdim + vb * 64, p.proj_ld, nt, d.vdim - vb * 64, nullptr, 1.0f, linear);
     __syncthreads();
     float acc[8][4];
 #pragma unroll
@@ -362,7 +511,7 @@ static __global__ void __launch_bounds__(128) mem_chunk_kernel(const __grid_cons
         }
     }
     if (vb == 0) {
-        for (int i = tid; i < 64 && kb * 64 + i < d.dim; i += 128) {
+        for (int i = tid; i < 64 && kb * 64 + i < d.dim && !linear; i += 128) {
             float s = 0.0f;
             for (int t = 0; t < nt; ++t) s += Elem<__nv_bfloat16>::to_f32(kh[t * MEM_LD + i]) + Elem<__nv_bfloat16>::to_f32(kl[t * MEM_LD + i]);
             p.UN[((size_t)c * d.H + h) * d.dim + kb * 64 + i] = s;
@@ -370,7 +519,7 @@ static __global__ void __launch_bounds__(128) mem_chunk_kernel(const __grid_cons
         if (kb == 0 && tid == 0) {
             p.gm[((size_t)c * d.H + h) * 2] = Fend;
             p.gm[((size_t)c * d.H + h) * 2 + 1] = wmax;
-            if (c == 0) p.m_live[h] = p.state[d.m_off() + h * d.nslice];
+            if (c == 0) p.m_live[h] = linear ? 0.0f : p.state[d.m_off() + h * d.nslice];
         }
     }
 }
@@ -401,6 +550,7 @@ static __global__ void __launch_bounds__(256) mem_scan_kernel(const __grid_const
         *S = s;
         return;
     }
+    if (d.linear()) return;
     float* nl = p.state + d.n_off() + (size_t)h * d.nslice * d.dim;
     for (int i = tid; i < d.dim; i += 256) {
         float mm = m, s = nl[i];
@@ -436,8 +586,11 @@ static __global__ void __launch_bounds__(128) mem_out_kernel(const __grid_consta
     __nv_bfloat16 *qh = t, *ql = t + MEM_TILE_ELEMS, *kh = t + 2 * MEM_TILE_ELEMS, *kl = t + 3 * MEM_TILE_ELEMS;
     __nv_bfloat16 *sh = t + 4 * MEM_TILE_ELEMS, *sl = t + 5 * MEM_TILE_ELEMS, *vh = t + 6 * MEM_TILE_ELEMS, *vl = t + 7 * MEM_TILE_ELEMS;
     mem_chunk_gates(p, h, t0, nt, F, I, &tmp);
-    const float m0 = m_start[(size_t)c * d.H + h];
-    if (tid < MEM_CHUNK) {  // M_t by an inclusive maximum scan
+    const bool linear = d.linear();
+    const float m0 = linear ? 0.0f : m_start[(size_t)c * d.H + h];
+    if (linear) {
+        if (tid < MEM_CHUNK) Mx[tid] = -F[tid];
+    } else if (tid < MEM_CHUNK) {  // M_t by an inclusive maximum scan
         float a = I[tid] - F[tid];
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
@@ -448,12 +601,12 @@ static __global__ void __launch_bounds__(128) mem_out_kernel(const __grid_consta
         Mx[tid] = fmaxf(a, m0);
     }
     __syncthreads();
-    if (tid >= 32 && tid < MEM_CHUNK) Mx[tid] = fmaxf(Mx[tid], tmp);
+    if (tid >= 32 && tid < MEM_CHUNK && !linear) Mx[tid] = fmaxf(Mx[tid], tmp);
     const float* row0 = p.proj + (size_t)t0 * p.proj_ld;
     const float* S0 = p.U + ((size_t)c * d.H + h) * d.dim * d.vs;
     const float* N0 = p.UN + ((size_t)c * d.H + h) * d.dim;
-    const float qscale = 1.0f / sqrtf((float)d.dim);
-    mem_load_tile(vh, vl, row0 + p.pl.rv + h * d.vdim + vb * 64, p.proj_ld, nt, d.vdim - vb * 64, nullptr, 1.0f);
+    const float qscale = linear ? 1.0f : 1.0f / sqrtf((float)d.dim);
+    mem_load_tile(vh, vl, row0 + p.pl.rv + h * d.vdim + vb * 64, p.proj_ld, nt, d.vdim - vb * 64, nullptr, 1.0f, linear);
     float sc[8][4], o[8][4], nq = 0.0f;
 #pragma unroll
     for (int i = 0; i < 8; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
@@ -461,11 +614,11 @@ static __global__ void __launch_bounds__(128) mem_out_kernel(const __grid_consta
     const uint32_t b_off = (uint32_t)((lane & 7) + 8 * (lane >> 4)) * (MEM_LD * 2) + (uint32_t)((lane >> 3) & 1) * 16u;
     for (int kb = 0; kb * 64 < d.dim; ++kb) {
         __syncthreads();  // the previous block's tiles are no longer read
-        mem_load_tile(qh, ql, row0 + p.pl.rq + h * d.dim + kb * 64, p.proj_ld, nt, d.dim - kb * 64, nullptr, qscale);
-        mem_load_tile(kh, kl, row0 + p.pl.rk + h * d.dim + kb * 64, p.proj_ld, nt, d.dim - kb * 64, nullptr, 1.0f);
+        mem_load_tile(qh, ql, row0 + p.pl.rq + h * d.dim + kb * 64, p.proj_ld, nt, d.dim - kb * 64, nullptr, qscale, linear);
+        mem_load_tile(kh, kl, row0 + p.pl.rk + h * d.dim + kb * 64, p.proj_ld, nt, d.dim - kb * 64, nullptr, 1.0f, linear);
         mem_load_tile(sh, sl, S0 + (size_t)kb * 64 * d.vs + vb * 64, d.vs, d.dim - kb * 64, d.vdim - vb * 64, nullptr, 1.0f);
         __syncthreads();
-        {   // n_0 . q: two threads per token
+        if (!linear) {   // n_0 . q: two threads per token
             const int tt = tid >> 1, i0 = (tid & 1) * 32;
             for (int i = i0; i < i0 + 32 && kb * 64 + i < d.dim; ++i)
                 nq = fmaf(Elem<__nv_bfloat16>::to_f32(qh[tt * MEM_LD + i]) + Elem<__nv_bfloat16>::to_f32(ql[tt * MEM_LD + i]), N0[kb * 64 + i], nq);
@@ -522,8 +675,8 @@ static __global__ void __launch_bounds__(128) mem_out_kernel(const __grid_consta
         al[0] = pack2<B>(s0[0] - round16<B>(s0[0]), s0[1] - round16<B>(s0[1])); al[1] = pack2<B>(s0[2] - round16<B>(s0[2]), s0[3] - round16<B>(s0[3]));
         al[2] = pack2<B>(s1[0] - round16<B>(s1[0]), s1[1] - round16<B>(s1[1])); al[3] = pack2<B>(s1[2] - round16<B>(s1[2]), s1[3] - round16<B>(s1[3]));
     });
-    const float d_a = 1.0f / (fmaxf(fabsf(n_a + e_a * NQ[ta]), expf(-(F[ta] + M_a))) + 1e-6f);
-    const float d_b = 1.0f / (fmaxf(fabsf(n_b + e_b * NQ[tb]), expf(-(F[tb] + M_b))) + 1e-6f);
+    const float d_a = linear ? 1.0f : 1.0f / (fmaxf(fabsf(n_a + e_a * NQ[ta]), expf(-(F[ta] + M_a))) + 1e-6f);
+    const float d_b = linear ? 1.0f : 1.0f / (fmaxf(fabsf(n_b + e_b * NQ[tb]), expf(-(F[tb] + M_b))) + 1e-6f);
     const int ld = d.H * d.vdim;
 #pragma unroll
     for (int n = 0; n < 8; ++n) {
@@ -538,20 +691,27 @@ static __global__ void __launch_bounds__(128) mem_out_kernel(const __grid_consta
     }
 }
 
-// per token: each head's read-out divided by its root mean square, times norm weight and gate, as a GEMM operand
+// per token: the read-outs, each head divided by its root mean square (linear attention: all heads by their common one),
+// times norm weight and gate, as a GEMM operand
 template <typename AT>
 __global__ void __launch_bounds__(256) mem_rows_kernel(const float* __restrict__ mem, const float* __restrict__ proj, int proj_ld, int gate_off, MemDims d,
                                                        const float* __restrict__ norm, AT* __restrict__ hi, AT* __restrict__ lo, int ld) {
+    __shared__ float red[32];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, n = d.H * d.vdim;
     const float* row = mem + (size_t)blockIdx.x * n;
     const float* gate = proj + (size_t)blockIdx.x * proj_ld + gate_off;
-    for (int h = warp; h < d.H; h += 8) {
+    auto put = [&](int j, float r) { pf_store(hi, lo, (size_t)blockIdx.x * ld + j, row[j] * r * norm[j] * sigmoid(gate[j])); };
+    if (d.linear()) {
         float ss = 0.0f;
-        for (int i = lane; i < d.vdim; i += 32) { const float v = row[h * d.vdim + i]; ss = fmaf(v, v, ss); }
-        const float r = 1.0f / sqrtf(warp_sum(ss) / (float)d.vdim + d.eps);
-        for (int i = lane; i < d.vdim; i += 32) {
-            const int j = h * d.vdim + i;
-            pf_store(hi, lo, (size_t)blockIdx.x * ld + j, row[j] * r * norm[j] * sigmoid(gate[j]));
+        for (int j = threadIdx.x; j < n; j += 256) ss = fmaf(row[j], row[j], ss);
+        const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)n + d.eps);
+        for (int j = threadIdx.x; j < n; j += 256) put(j, r);
+    } else {
+        for (int h = warp; h < d.H; h += 8) {
+            float ss = 0.0f;
+            for (int i = lane; i < d.vdim; i += 32) { const float v = row[h * d.vdim + i]; ss = fmaf(v, v, ss); }
+            const float r = 1.0f / sqrtf(warp_sum(ss) / (float)d.vdim + d.eps);
+            for (int i = lane; i < d.vdim; i += 32) put(h * d.vdim + i, r);
         }
     }
     for (int j = n + threadIdx.x; j < ld; j += 256) pf_store(hi, lo, (size_t)blockIdx.x * ld + j, 0.0f);
@@ -582,31 +742,68 @@ __global__ void __launch_bounds__(256) parallel_mix_rows_kernel(float* __restric
     }
 }
 
-// y: one row per token, or (slots != nullptr) the rows of the token's chosen experts, weighted by their scores in the
-// order they were chosen
-template <typename AT>
-__global__ void __launch_bounds__(256) normed_residual_rows_kernel(float* __restrict__ x, const float* __restrict__ y, int y_ld, const int* __restrict__ slots,
-                                                                   const float* __restrict__ weights, int top, const float* __restrict__ gain, float mult, float eps,
-                                                                   int D, AT* __restrict__ hi, AT* __restrict__ lo) {
-    extern __shared__ float sum[];  // [D]
-    __shared__ float red[32];
-    float ss = 0.0f;
-    for (int i = threadIdx.x; i < D; i += 256) {
-        float v = 0.0f;
-        if (slots != nullptr) {
-            for (int k = 0; k < top; ++k) v = fmaf(weights[blockIdx.x * top + k], y[(size_t)slots[blockIdx.x * top + k] * y_ld + i], v);
-        } else {
-            v = y[(size_t)blockIdx.x * y_ld + i];
-        }
-        sum[i] = v;
-        ss = fmaf(v, v, ss);
+// mean and reciprocal deviation of a row in shared memory
+__device__ inline void row_moments(const float* row, int D, int kind, float eps, float* red, float& mean, float& r) {
+    mean = 0.0f;
+    if (kind == VecNorm::LAYER) {
+        float s = 0.0f;
+        for (int i = threadIdx.x; i < D; i += 256) s += row[i];
+        mean = block_sum(s, red) * (1.0f / (float)D);
     }
-    const float r = mult / sqrtf(block_sum(ss, red) * (1.0f / (float)D) + eps);
-    for (int i = threadIdx.x; i < D; i += 256) {
-        const size_t at = (size_t)blockIdx.x * D + i;
-        const float v = x[at] + sum[i] * r * gain[i];
-        x[at] = v;
-        pf_store(hi, lo, at, v);
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < D; i += 256) { const float v = row[i] - mean; ss = fmaf(v, v, ss); }
+    r = 1.0f / sqrtf(block_sum(ss, red) * (1.0f / (float)D) + eps);
+}
+
+// x += mult * post(y) + add, and pre(x) as a GEMM operand (InResidual, mixers.cuh).  y: none, one row per token, or (slots !=
+// nullptr) the rows of the token's chosen experts, weighted by their scores in the order they were chosen
+struct ResidualRows {
+    float* x;
+    const float* y;
+    int y_ld;
+    const int* slots;
+    const float* weights;
+    int top;
+    VecNorm post;
+    const float* add;
+    VecNorm pre;
+    float mult, eps;
+    int D;
+};
+template <typename AT>
+__global__ void __launch_bounds__(256) residual_rows_kernel(ResidualRows p, AT* __restrict__ hi, AT* __restrict__ lo) {
+    extern __shared__ float sum[];  // [D]; a thread touches its own entries only
+    __shared__ float red[32];
+    float mean = 0.0f, r = 1.0f;
+    const bool normed = p.y != nullptr && p.post.kind != VecNorm::NONE;
+    if (p.y != nullptr) {
+        for (int i = threadIdx.x; i < p.D; i += 256) {
+            float v = 0.0f;
+            if (p.slots != nullptr) {
+                for (int k = 0; k < p.top; ++k) v = fmaf(p.weights[blockIdx.x * p.top + k], p.y[(size_t)p.slots[blockIdx.x * p.top + k] * p.y_ld + i], v);
+            } else {
+                v = p.y[(size_t)blockIdx.x * p.y_ld + i];
+            }
+            sum[i] = v;
+        }
+        if (normed) row_moments(sum, p.D, p.post.kind, p.eps, red, mean, r);
+    }
+    r *= p.mult;
+    for (int i = threadIdx.x; i < p.D; i += 256) {
+        const size_t at = (size_t)blockIdx.x * p.D + i;
+        float v = p.x[at];
+        if (normed) v += (sum[i] - mean) * r * p.post.w[i] + (p.post.b != nullptr ? p.mult * p.post.b[i] : 0.0f);
+        else if (p.y != nullptr) v += sum[i] * r;
+        if (p.add != nullptr) v += p.add[i];
+        p.x[at] = v;
+        sum[i] = v;
+    }
+    const bool ahead = p.pre.kind != VecNorm::NONE;
+    if (ahead) row_moments(sum, p.D, p.pre.kind, p.eps, red, mean, r);
+    for (int i = threadIdx.x; i < p.D; i += 256) {
+        float v = sum[i];
+        if (ahead) v = (v - mean) * r * p.pre.w[i] + (p.pre.b != nullptr ? p.pre.b[i] : 0.0f);
+        pf_store(hi, lo, (size_t)blockIdx.x * p.D + i, v);
     }
 }
 

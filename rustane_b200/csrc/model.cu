@@ -403,9 +403,15 @@ int cd_can_rewind(const cd_model* m, size_t len) {
     return !m->family->can_rewind || m->family->can_rewind(m, len) ? 1 : 0;
 }
 
+// calls that start from a hidden state instead of a token id
+static int hidden_input_guard(cd_model* m) {
+    return m->needs_token ? fail(m, CD_ERR_UNSUPPORTED, "this model's layers read the token id: use the calls that take one") : (int)CD_OK;
+}
+
 int cd_decode_token(cd_model* m, const float* x_in, float* x_out) {
     if (m) { int g_ = tp_guard(m, false); if (g_) return g_; }
     if (!m || !x_in || !x_out) return fail(m, CD_ERR_INVALID, "null argument");
+    if (int g_ = hidden_input_guard(m)) return g_;
     int rc = check_room(m, 1);
     if (rc) return rc;
     CK(m, cudaMemcpyAsync(m->x_a, x_in, (size_t)m->cfg.dim * 4, cudaMemcpyHostToDevice, m->stream));
@@ -453,6 +459,7 @@ static int argmax_common(cd_model* m, int input, uint32_t token, uint32_t* out) 
 
 int cd_decode_token_argmax(cd_model* m, const float* x_in, uint32_t* out) {
     if (!m || !x_in || !out) return fail(m, CD_ERR_INVALID, "null argument");
+    if (int g_ = hidden_input_guard(m)) return g_;
     int rc = check_room(m, 1);
     if (rc) return rc;
     CK(m, cudaMemcpyAsync(m->x_a, x_in, (size_t)m->cfg.dim * 4, cudaMemcpyHostToDevice, m->stream));

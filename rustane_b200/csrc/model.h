@@ -111,6 +111,7 @@ struct cd_model {
     cd_hybrid_state* hybrid = nullptr;  // set: the handle is a configured decoder (hybrid.h)
     bool replicated_head = false;       // several ranks, each with the whole LM head (expert parallelism)
     float rms_eps = cd::RMS_EPS;        // of the norm ahead of the LM head
+    bool needs_token = false;           // layers read the token itself: a hidden state alone cannot be stepped
     size_t state_len = 0;               // tokens the recurrent state has seen (families that keep one); SIZE_MAX: unknown
     cd_moe_state* moe = nullptr;  // set: the handle is a MoE + MLA decoder
     cd_config cfg;       // what this GPU holds: under tensor parallelism heads, kv_heads, hidden, q_dim, kv_dim are per rank

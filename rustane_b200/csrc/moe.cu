@@ -7,7 +7,7 @@
 #include <vector>
 
 #include "step.cuh"
-#include "moe.cuh"
+#include "latent_launch.cuh"
 
 using namespace cd;
 
@@ -102,22 +102,13 @@ cudaError_t enqueue_step_moe_t(cd_model* m, const cd_step& p) {
         count_launch(m);
         TRY(cudaGetLastError());
     }
-    const MlaDims md{c.heads, mc.kv_latent, mc.rope_dim, mc.nope_dim, mc.v_dim, m->page_tokens};
+    const MlaDims md{c.heads, mc.kv_latent, mc.rope_dim, mc.nope_dim, mc.v_dim, m->page_tokens, mc.kv_latent, mc.rope_dim, mc.nope_dim, mc.rope_dim, 0, RMS_EPS};
     const MoeDims ed{c.dim, c.hidden, S.shared_cols};
     const MoePick pick{S.loc_ids, S.loc_w, S.n_loc};
     const int W = mc.kv_latent + mc.rope_dim, QA = c.q_dim + W, units = mc.top_k * c.hidden + S.shared_cols;
     const bool ep = m->tp_world > 1;
     const float scale = 1.0f / std::sqrt((float)c.hd);
-    // the tensor-core attention takes a 16-bit cache of the 512-wide latent geometry; anything else the plain kernel
-    const bool attn_mma = !std::is_same<KT, float>::value && mc.kv_latent == MLA_MMA_C && W % 16 == 0 && c.heads <= 16;
-    const size_t attn_smem = attn_mma ? mla_mma_smem_bytes(W)
-                                      : ((size_t)(c.heads + MLA_TILE) * (W + 1) + (size_t)c.heads * MLA_TILE + 3 * c.heads) * sizeof(float);
-    static size_t attn_set = 0, w2_set = 0;  // per instantiation
-    if (attn_smem > attn_set) {
-        if constexpr (!std::is_same<KT, float>::value) TRY(cudaFuncSetAttribute(mla_attn_mma_kernel<KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)std::max(attn_smem, mla_mma_smem_bytes(W))));
-        TRY(cudaFuncSetAttribute(mla_attn_kernel<KT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)attn_smem));
-        attn_set = attn_smem;
-    }
+    static size_t w2_set = 0;  // per instantiation
     if (!S.stream_ffn && (size_t)units * 4 > w2_set) {
         TRY(cudaFuncSetAttribute(moe_w2_kernel<WT>, cudaFuncAttributeMaxDynamicSharedMemorySize, units * 4));
         w2_set = (size_t)units * 4;
@@ -130,19 +121,8 @@ cudaError_t enqueue_step_moe_t(cd_model* m, const cd_step& p) {
         if (ep && l > 0) { m->tp_in.in_reduce = l; m->tp_in.res = m->x_b; m->tp_in.x_out = m->x_a; }  // x = x2 + alpha * sum(ranks' FFN partials)
         TRY((launch_gemv<WT, 1, true>(m, L.wqa, m->x_a, L.gamma1, nullptr, QA, c.dim, EpiStore{S.qa})));
         m->cur_cls = CLS_ATTN;
-        TRY(launch_chain(m, mla_post_kernel<WT, KT>, dim3((c.heads * mc.kv_latent + 127) / 128 + 1), dim3(128), std::max(c.heads * mc.nope_dim, mc.kv_latent) * sizeof(float),
-                         (const float*)S.qa, (const WT*)L.wuk_t, (const float*)L.gamma_kv, (const float2*)m->rope, (const int*)m->page_table, (const DevState*)m->st,
-                         (KT*)m->layers[l].kv, S.qabs, attn_mma ? (KT*)S.qsplit : (KT*)nullptr, md));
-        if constexpr (!std::is_same<KT, float>::value) {
-            if (attn_mma)
-                TRY(launch_chain(m, mla_attn_mma_kernel<KT>, dim3(S.nsplit), dim3(MLA_MMA_THREADS), attn_smem, (const KT*)S.qsplit, (const KT*)m->layers[l].kv,
-                                 (const int*)m->page_table, (const DevState*)m->st, S.part_acc, S.part_ml, md, S.nsplit, scale, &m->st->error));
-        }
-        if (!attn_mma)
-            TRY(launch_chain(m, mla_attn_kernel<KT>, dim3(S.nsplit), dim3(256), attn_smem, (const float*)S.qabs, (const KT*)m->layers[l].kv, (const int*)m->page_table,
-                             (const DevState*)m->st, S.part_acc, S.part_ml, md, S.nsplit, scale));
-        TRY(launch_chain(m, mla_out_kernel<WT>, dim3(c.heads, (mc.v_dim + 31) / 32), dim3(256), (mc.kv_latent + S.nsplit) * sizeof(float), (const float*)S.part_acc,
-                         (const float*)S.part_ml, (const WT*)L.wuv_t, m->attn, (const DevState*)m->st, md, S.nsplit, attn_mma ? MLA_MMA_TILE : MLA_TILE));
+        TRY((launch_mla<WT, KT>(m, MlaStep{md, S.qa, L.wuk_t, L.wuv_t, L.gamma_kv, Rotation{m->rope, nullptr, mc.rope_dim}, m->layers[l].kv, S.qabs, S.qsplit,
+                                           S.part_acc, S.part_ml, m->attn, S.nsplit, scale})));
         m->cur_cls = CLS_WO;
         TRY((launch_gemv<WT, 1, false>(m, L.wo, m->attn, nullptr, nullptr, c.dim, c.heads * mc.v_dim, EpiResidual{m->x_a, m->x_b, m->alpha})));
         m->cur_cls = CLS_W13;

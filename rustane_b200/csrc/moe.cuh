@@ -24,7 +24,8 @@
 
 namespace cd {
 
-constexpr int MLA_MAX_HEADS = 16;   // heads whose state one attention thread keeps
+constexpr int MLA_MAX_HEADS = 16;   // heads whose state one attention CTA keeps: more heads go to further CTAs
+constexpr int MLA_MAX_COLS = 512;   // latent columns it accumulates: wider latents likewise
 constexpr int MLA_TILE = 16;        // cached positions per attention tile
 
 // dot of one weight row (K elements, storage WT) with x (fp32, shared memory): the lanes of a warp take
@@ -77,8 +78,47 @@ __device__ inline void warp_rows_dot(const WT* __restrict__ rows, size_t stride,
     for (int r = 0; r < NR; ++r) out[r] = warp_sum(a[r]);
 }
 
+// Widths as stored: the cache row is [latent | rope], a row of the absorbed-key matrix has nope elements (each a multiple of
+// 16 bytes where the kernels ask for it, zeros behind the model's own widths latent_n, rope_n, nope_n, which are those of
+// the projection row [heads (nope_n + rope_n) | latent_n | rope_n]).
 struct MlaDims {
     int heads, latent, rope, nope, vdim, page_tokens;
+    int latent_n, rope_n, nope_n;
+    int rot_dims;        // rotated entries of the rope part, the first ones
+    int window;          // positions seen, itself included; 0: all
+    float eps;           // of the latent's norm
+    __host__ __device__ int row() const { return latent + rope; }
+    __host__ __device__ int head_blocks() const { return (heads + MLA_MAX_HEADS - 1) / MLA_MAX_HEADS; }
+    __host__ __device__ int col_blocks() const { return (latent + MLA_MAX_COLS - 1) / MLA_MAX_COLS; }
+    // the attention kernels' split of the visible positions: slice s holds first .. first + per - 1 (up to pos)
+    __device__ int first_seen(int pos) const { return window > 0 ? max(0, pos - window + 1) : 0; }
+    __device__ int slice(int pos, int nsplit, int tile) const {
+        const int per = (pos + 1 - first_seen(pos) + nsplit - 1) / nsplit;
+        return (per + tile - 1) / tile * tile;
+    }
+};
+
+// cos and sin of a position's k-th rotation: from a table [position][dims / 2], or worked out from the angular frequencies
+// (angle and its reduction in double, so that far positions keep their fp32 accuracy)
+struct Rotation {
+    const float2* table;
+    const double* freq;
+    int dims;
+    __device__ float2 at(int pos, int k) const {
+        if (table != nullptr) return table[(size_t)pos * (dims / 2) + k];
+        const double turns = (double)pos * freq[k] * 0.15915494309189533577;  // 1 / (2 pi)
+        const float a = (float)((turns - rint(turns)) * 6.283185307179586477);
+        float2 cs;
+        sincosf(a, &cs.y, &cs.x);
+        return cs;
+    }
+    // entry d of a vector whose raw entries get(i) returns
+    template <class Get> __device__ float entry(int pos, int d, Get get) const {
+        if (d >= dims) return get(d);
+        const float2 cs = at(pos, d >> 1);
+        const float u = get(d & ~1), v = get(d | 1);
+        return (d & 1) ? v * cs.x + u * cs.y : u * cs.x - v * cs.y;
+    }
 };
 
 // ---------------------------------------------------------------------- after the q | latent | key GEMV
@@ -88,22 +128,23 @@ struct MlaDims {
 // [rmsnorm(latent) | rope(key)].  qabs[h] = [q'_h (C) | rope(q_rope_h) (R)].
 template <typename WT, typename KT>
 __global__ void __launch_bounds__(128)
-mla_post_kernel(const float* __restrict__ qa, const WT* __restrict__ wuk_t, const float* __restrict__ gamma_kv, const float2* __restrict__ rope,
+mla_post_kernel(const float* __restrict__ qa, const WT* __restrict__ wuk_t, const float* __restrict__ gamma_kv, Rotation rot,
                 const int* __restrict__ page_table, const DevState* st, KT* __restrict__ lat_pool, float* __restrict__ qabs, KT* __restrict__ qsplit,
                 MlaDims d) {
     extern __shared__ float sm[];  // [heads * N] the no-position parts of q (absorb CTAs) or [C] the raw latent (last CTA)
     __shared__ float red[32];
     constexpr int EPC = Elem<WT>::EPC;
     const int tid = threadIdx.x;
-    const int H = d.heads, C = d.latent, R = d.rope, N = d.nope, QH = N + R;
-    // qsplit (16-bit cache only): [2][16][C + R], the 16-bit head of qabs and the 16-bit remainder, the tensor-core
-    // attention's A operand
+    const int H = d.heads, C = d.latent, R = d.rope, N = d.nope, QH = d.nope_n + d.rope_n;
+    // qsplit (16-bit cache only): per block of 16 heads [2][16][C + R], the 16-bit head of qabs and the 16-bit remainder, the
+    // tensor-core attention's A operand
     auto put = [&](int h, int k, float v) {
         qabs[(size_t)h * (C + R) + k] = v;
         if (qsplit != nullptr) {
+            KT* q = qsplit + (size_t)((h >> 4) * 32 + (h & 15)) * (C + R) + k;
             const KT hi = Elem<KT>::from_f32(v);
-            qsplit[(size_t)h * (C + R) + k] = hi;
-            qsplit[(size_t)(16 + h) * (C + R) + k] = Elem<KT>::from_f32(v - Elem<KT>::to_f32(hi));
+            *q = hi;
+            q[(size_t)16 * (C + R)] = Elem<KT>::from_f32(v - Elem<KT>::to_f32(hi));
         }
     };
     if (blockIdx.x + 1 < gridDim.x) {
@@ -115,11 +156,13 @@ mla_post_kernel(const float* __restrict__ qa, const WT* __restrict__ wuk_t, cons
         for (int j = 0; j < PRE; ++j) w[j] = j < N / EPC ? ldg_stream(row + (size_t)j * 16) : make_uint4(0, 0, 0, 0);
         pdl_wait();  // the weights above do not depend on the previous kernel, q does
         pdl_launch_dependents();
-        for (int i = tid; i < H * N; i += blockDim.x) sm[i] = __ldcg(qa + (size_t)(i / N) * QH + (i % N));
+        // only the heads this CTA's rows belong to
+        const int h0 = (int)(blockIdx.x * blockDim.x) / C, h1 = min((int)((blockIdx.x + 1) * blockDim.x - 1) / C, H - 1);
+        for (int i = tid; i < (h1 - h0 + 1) * N; i += blockDim.x) sm[i] = i % N < d.nope_n ? __ldcg(qa + (size_t)(h0 + i / N) * QH + (i % N)) : 0.0f;
         __syncthreads();
         if ((int)(blockIdx.x * blockDim.x) + tid >= H * C) return;
         const int h = r / C;
-        const float* qn = sm + h * N;
+        const float* qn = sm + (h - h0) * N;
         float acc = 0.0f;
 #pragma unroll
         for (int j = 0; j < PRE; ++j) {
@@ -150,46 +193,46 @@ mla_post_kernel(const float* __restrict__ qa, const WT* __restrict__ wuk_t, cons
     pdl_wait();
     pdl_launch_dependents();
     const int pos = __ldcg(&st->pos);
-    for (int i = tid; i < H * (R / 2); i += blockDim.x) {  // RoPE on q's RoPE parts
-        const int h = i / (R / 2), k = i % (R / 2);
-        const float e = __ldcg(qa + (size_t)h * QH + N + 2 * k), o = __ldcg(qa + (size_t)h * QH + N + 2 * k + 1);
-        const float2 cs = rope[(size_t)pos * (R / 2) + k];
-        put(h, C + 2 * k, e * cs.x - o * cs.y);
-        put(h, C + 2 * k + 1, o * cs.x + e * cs.y);
+    for (int i = tid; i < H * R; i += blockDim.x) {  // rotation of q's part of it
+        const int h = i / R, k = i % R;
+        const float* q = qa + (size_t)h * QH + d.nope_n;
+        put(h, C + k, k < d.rope_n ? rot.entry(pos, k, [&](int j) { return __ldcg(q + j); }) : 0.0f);
     }
-    // the cache row: rmsnorm(latent) | rope(key)
+    // the cache row: normed latent | rotated key
     const float* craw = qa + (size_t)H * QH;
     float ss = 0.0f;
-    for (int i = tid; i < C; i += blockDim.x) {
+    for (int i = tid; i < d.latent_n; i += blockDim.x) {
         const float v = __ldcg(craw + i);
         sm[i] = v;
         ss += v * v;
     }
     const float tot = block_sum(ss, red);
-    const float inv = 1.0f / sqrtf(tot * (1.0f / (float)C) + RMS_EPS);
+    const float inv = 1.0f / sqrtf(tot * (1.0f / (float)d.latent_n) + d.eps);
     const int page = page_table[pos / d.page_tokens], off = pos % d.page_tokens;
     KT* row = lat_pool + ((size_t)page * d.page_tokens + off) * (C + R);
-    for (int i = tid; i < C; i += blockDim.x) row[i] = Elem<KT>::from_f32(sm[i] * inv * gamma_kv[i]);
-    for (int i = tid; i < R / 2; i += blockDim.x) {
-        const float e = __ldcg(craw + C + 2 * i), o = __ldcg(craw + C + 2 * i + 1);
-        const float2 cs = rope[(size_t)pos * (R / 2) + i];
-        row[C + 2 * i] = Elem<KT>::from_f32(e * cs.x - o * cs.y);
-        row[C + 2 * i + 1] = Elem<KT>::from_f32(o * cs.x + e * cs.y);
-    }
+    for (int i = tid; i < C; i += blockDim.x) row[i] = Elem<KT>::from_f32(i < d.latent_n ? sm[i] * inv * gamma_kv[i] : 0.0f);
+    for (int i = tid; i < R; i += blockDim.x)
+        row[C + i] = Elem<KT>::from_f32(i < d.rope_n ? rot.entry(pos, i, [&](int j) { return __ldcg(craw + d.latent_n + j); }) : 0.0f);
 }
+__host__ __device__ inline size_t mla_post_smem_floats(const MlaDims& d) { return max((128 / d.latent + 2) * d.nope, d.latent); }
 
 // ---------------------------------------------------------------------- latent attention, one slice of cached positions per CTA
 // score_h(t) = qabs_h . row(t) * scale over the C + R wide cache row; out_h = sum_t p_h(t) row(t)[0 .. C).
 // Shared memory: qs [H][W + 1], rows [MLA_TILE][W + 1] (W = C + R; the pad keeps the columns on
 // different banks), sc [H][MLA_TILE], state [3][H].  256 threads; thread t owns latent dimensions
-// t and t + 256 of every head.
+// t and t + 256 of every head.  grid = (slices, blocks of 16 heads, blocks of 512 latent columns).
+__host__ __device__ inline size_t mla_attn_smem_floats(const MlaDims& d) {
+    const size_t h = min(d.heads, MLA_MAX_HEADS), w = d.row();
+    return h * (w + 1) + (size_t)MLA_TILE * (w + 1) + h * MLA_TILE + 3 * h;
+}
 template <typename KT>
 __global__ void __launch_bounds__(256)
 mla_attn_kernel(const float* __restrict__ qabs, const KT* __restrict__ lat_pool, const int* __restrict__ page_table, const DevState* st,
                 float* __restrict__ part_acc, float* __restrict__ part_ml, MlaDims d, int nsplit, float scale) {
     extern __shared__ float sm[];
     constexpr float NEG = -3.402823466e+38f;
-    const int tid = threadIdx.x, H = d.heads, C = d.latent, W = d.latent + d.rope, LD = W + 1, s = blockIdx.x;
+    const int h0 = blockIdx.y * MLA_MAX_HEADS, col0 = blockIdx.z * MLA_MAX_COLS;
+    const int tid = threadIdx.x, H = min(d.heads - h0, MLA_MAX_HEADS), C = min(d.latent - col0, MLA_MAX_COLS), W = d.latent + d.rope, LD = W + 1, s = blockIdx.x;
     float* qs = sm;                          // [H][LD]
     float* rows = qs + (size_t)H * LD;       // [MLA_TILE][LD]
     float* sc = rows + (size_t)MLA_TILE * LD;  // [H][MLA_TILE] probabilities of the tile
@@ -198,11 +241,9 @@ mla_attn_kernel(const float* __restrict__ qabs, const KT* __restrict__ lat_pool,
     float* corr = lrun + H;                  // [H] rescale factor of the tile
     pdl_wait();
     pdl_launch_dependents();  // after the wait: at most this kernel and the next one overlap
-    const int attn_len = __ldcg(&st->pos) + 1;
-    int per = (attn_len + nsplit - 1) / nsplit;
-    per = (per + MLA_TILE - 1) / MLA_TILE * MLA_TILE;
-    const int t0 = s * per, t1 = min(attn_len, t0 + per);
-    for (int i = tid; i < H * W; i += 256) qs[(i / W) * LD + (i % W)] = __ldcg(qabs + i);
+    const int pos = __ldcg(&st->pos), per = d.slice(pos, nsplit, MLA_TILE);
+    const int t0 = d.first_seen(pos) + s * per, t1 = min(pos + 1, t0 + per);
+    for (int i = tid; i < H * W; i += 256) qs[(i / W) * LD + (i % W)] = __ldcg(qabs + (size_t)h0 * W + i);
     if (tid < H) { mrun[tid] = NEG; lrun[tid] = 0.0f; }
     float acc[MLA_MAX_HEADS][2];
 #pragma unroll
@@ -259,8 +300,8 @@ mla_attn_kernel(const float* __restrict__ qabs, const KT* __restrict__ lat_pool,
                 float a0 = acc[h][0] * c, a1 = acc[h][1] * c;
                 for (int j = 0; j < nt; ++j) {
                     const float p = sc[h * MLA_TILE + j];
-                    if (tid < C) a0 = fmaf(p, rows[j * LD + tid], a0);
-                    if (tid + 256 < C) a1 = fmaf(p, rows[j * LD + tid + 256], a1);
+                    if (tid < C) a0 = fmaf(p, rows[j * LD + col0 + tid], a0);
+                    if (tid + 256 < C) a1 = fmaf(p, rows[j * LD + col0 + tid + 256], a1);
                 }
                 acc[h][0] = a0; acc[h][1] = a1;
             }
@@ -270,14 +311,14 @@ mla_attn_kernel(const float* __restrict__ qabs, const KT* __restrict__ lat_pool,
 #pragma unroll
     for (int h = 0; h < MLA_MAX_HEADS; ++h) {
         if (h < H) {
-            float* pa = part_acc + ((size_t)s * H + h) * C;
+            float* pa = part_acc + ((size_t)s * d.heads + h0 + h) * d.latent + col0;
             if (tid < C) pa[tid] = acc[h][0];
             if (tid + 256 < C) pa[tid + 256] = acc[h][1];
         }
     }
     if (tid < H) {
-        part_ml[((size_t)s * H + tid) * 2 + 0] = mrun[tid];
-        part_ml[((size_t)s * H + tid) * 2 + 1] = lrun[tid];
+        part_ml[((size_t)s * d.heads + h0 + tid) * 2 + 0] = mrun[tid];
+        part_ml[((size_t)s * d.heads + h0 + tid) * 2 + 1] = lrun[tid];
     }
 }
 
@@ -296,10 +337,8 @@ mla_out_kernel(const float* __restrict__ part_acc, const float* __restrict__ par
     pdl_wait();
     pdl_launch_dependents();  // after the wait: at most this kernel and the next one overlap
     // the attention kernel's split of this context: slices of `per` positions, the first `nsplit` of them hold any
-    const int attn_len = __ldcg(&st->pos) + 1;
-    int per = (attn_len + nsplit_max - 1) / nsplit_max;
-    per = (per + tile - 1) / tile * tile;
-    const int nsplit = (attn_len + per - 1) / per;
+    const int pos = __ldcg(&st->pos), per = d.slice(pos, nsplit_max, tile);
+    const int nsplit = (pos - d.first_seen(pos)) / per + 1;
     if (warp == 0) {
         float M = NEG;
         for (int s = lane; s < nsplit; s += 32) {
@@ -356,8 +395,9 @@ mla_out_kernel(const float* __restrict__ part_acc, const float* __restrict__ par
 // cache itself carries its storage rounding.  One CTA of four warps per slice of cached positions, 64
 // positions at a time: the tile's rows arrive by one bulk copy each (row stride padded by 16 bytes: ldmatrix
 // without bank conflicts); warp w scores positions 16 w .. 16 w + 15, then owns latent columns
-// 128 w .. 128 w + 127 of every head.  Geometry: 16-bit cache, C = 512, (C + R) % 16 == 0, heads <= 16.
-constexpr int MLA_MMA_TILE = 64, MLA_MMA_C = 512, MLA_MMA_THREADS = 128;
+// CW w .. CW w + CW - 1 of every head (CW = 128; 64 and 32 for narrower latents).  grid = (slices, blocks of 16 heads, blocks
+// of 4 CW latent columns).  Geometry: 16-bit cache, C and R multiples of 16.
+constexpr int MLA_MMA_TILE = 64, MLA_MMA_THREADS = 128;
 
 template <typename KT> struct Mma16;
 template <> struct Mma16<__half> {
@@ -387,14 +427,16 @@ __host__ __device__ inline size_t mla_mma_smem_bytes(int W) {
            + 3 * 16 * 4 + 16;                            // running max, sum, rescale; mbarrier
 }
 
-template <typename KT>
+template <typename KT, int CW>
 __global__ void __launch_bounds__(MLA_MMA_THREADS)
 mla_attn_mma_kernel(const KT* __restrict__ qsplit, const KT* __restrict__ lat_pool, const int* __restrict__ page_table, const DevState* st,
                     float* __restrict__ part_acc, float* __restrict__ part_ml, MlaDims d, int nsplit, float scale, int* err) {
     extern __shared__ __align__(128) unsigned char smraw[];
     constexpr float NEG = -3.402823466e+38f;
-    constexpr int T = MLA_MMA_TILE, C = MLA_MMA_C, LDS = T + 1, LDP = T + 8;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, H = d.heads, W = d.latent + d.rope, s = blockIdx.x;
+    constexpr int T = MLA_MMA_TILE, LDS = T + 1, LDP = T + 8;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, h0 = blockIdx.y * MLA_MAX_HEADS, H = min(d.heads - h0, MLA_MAX_HEADS), C = d.latent;
+    const int W = d.latent + d.rope, s = blockIdx.x, col0 = (blockIdx.z * 4 + warp) * CW;  // this warp's latent columns
+    qsplit += (size_t)blockIdx.y * 32 * W;
     const uint32_t LDB = (uint32_t)W * 2u + 16u;
     unsigned char* rows_p = smraw;                                   // [T][LDB]
     unsigned char* qh_p = rows_p + (size_t)T * LDB;                  // [16][LDB]
@@ -411,11 +453,9 @@ mla_attn_mma_kernel(const KT* __restrict__ qsplit, const KT* __restrict__ lat_po
 
     pdl_wait();
     pdl_launch_dependents();  // after the wait: at most this kernel and the next one overlap
-    const int attn_len = __ldcg(&st->pos) + 1;
-    int per = (attn_len + nsplit - 1) / nsplit;
-    per = (per + T - 1) / T * T;
-    const int t0 = s * per, t1 = min(attn_len, t0 + per);
-    if (t0 >= t1) return;  // a slice past the context: mla_out_kernel merges ceil(attn_len / per) slices only
+    const int pos = __ldcg(&st->pos), per = d.slice(pos, nsplit, T);
+    const int t0 = d.first_seen(pos) + s * per, t1 = min(pos + 1, t0 + per);
+    if (t0 >= t1) return;  // a slice past the context: mla_out_kernel merges the slices that hold positions only
     if (tid == 0) {
         mbar_init(bar, 1);
         mbar_fence_init();
@@ -434,9 +474,9 @@ mla_attn_mma_kernel(const KT* __restrict__ qsplit, const KT* __restrict__ lat_po
         }
     };
     if (warp == 0) fetch(t0, true);
-    float acc[16][4];  // columns 128 warp + 8 nb + 2 (lane % 4) + {0, 1} of heads lane / 4 and lane / 4 + 8
+    float acc[CW / 8][4];  // columns col0 + 8 nb + 2 (lane % 4) + {0, 1} of heads lane / 4 and lane / 4 + 8
 #pragma unroll
-    for (int nb = 0; nb < 16; ++nb) acc[nb][0] = acc[nb][1] = acc[nb][2] = acc[nb][3] = 0.0f;
+    for (int nb = 0; nb < CW / 8; ++nb) acc[nb][0] = acc[nb][1] = acc[nb][2] = acc[nb][3] = 0.0f;
     const int g = lane >> 2, tq = lane & 3;
     uint32_t phase = 0;
     for (int tb = t0; tb < t1; tb += T) {
@@ -507,20 +547,21 @@ mla_attn_mma_kernel(const KT* __restrict__ qsplit, const KT* __restrict__ lat_po
             }
         }
         __syncthreads();
-        // ---- O += P V over this warp's 128 latent columns
+        // ---- O += P V over this warp's latent columns
         {
             const float ca = corr[g], cb = corr[g + 8];
 #pragma unroll
-            for (int nb = 0; nb < 16; ++nb) { acc[nb][0] *= ca; acc[nb][1] *= ca; acc[nb][2] *= cb; acc[nb][3] *= cb; }
+            for (int nb = 0; nb < CW / 8; ++nb) { acc[nb][0] *= ca; acc[nb][1] *= ca; acc[nb][2] *= cb; acc[nb][3] *= cb; }
             const uint32_t a_off = (uint32_t)(lane & 15) * (uint32_t)(LDP * 2) + (uint32_t)(lane >> 4) * 16u;
-            const uint32_t v_off = (uint32_t)((lane & 7) + 8 * ((lane >> 3) & 1)) * LDB + (uint32_t)(128 * warp + 8 * (lane >> 4)) * 2u;
+            const uint32_t v_off = (uint32_t)((lane & 7) + 8 * ((lane >> 3) & 1)) * LDB + (uint32_t)(col0 + 8 * (lane >> 4)) * 2u;
             for (int ks = 0; ks < T / 16; ++ks) {
                 if (16 * ks >= nt) break;
                 uint32_t ah[4], al[4];
                 ldsm_x4(ah, pha + a_off + (uint32_t)ks * 32u);
                 ldsm_x4(al, pla + a_off + (uint32_t)ks * 32u);
 #pragma unroll
-                for (int np = 0; np < 8; ++np) {
+                for (int np = 0; np < CW / 16; ++np) {
+                    if (col0 + 16 * np >= C) break;
                     uint32_t b[4];
                     ldsm_x4_trans(b, rows + v_off + (uint32_t)(16 * ks) * LDB + (uint32_t)np * 32u);
                     Mma16<KT>::mma(acc[2 * np], ah, b[0], b[1]);
@@ -534,14 +575,16 @@ mla_attn_mma_kernel(const KT* __restrict__ qsplit, const KT* __restrict__ lat_po
         if (warp == 0 && tb + T < t1) fetch(tb + T, false);
     }
 #pragma unroll
-    for (int nb = 0; nb < 16; ++nb) {
-        const int col = 128 * warp + 8 * nb + 2 * tq;
-        if (g < H) *reinterpret_cast<float2*>(part_acc + ((size_t)s * H + g) * C + col) = make_float2(acc[nb][0], acc[nb][1]);
-        if (g + 8 < H) *reinterpret_cast<float2*>(part_acc + ((size_t)s * H + g + 8) * C + col) = make_float2(acc[nb][2], acc[nb][3]);
+    for (int nb = 0; nb < CW / 8; ++nb) {
+        const int col = col0 + 8 * nb + 2 * tq;
+        if (col >= C) break;
+        float* pa = part_acc + ((size_t)s * d.heads + h0 + g) * C + col;
+        if (g < H) *reinterpret_cast<float2*>(pa) = make_float2(acc[nb][0], acc[nb][1]);
+        if (g + 8 < H) *reinterpret_cast<float2*>(pa + (size_t)8 * C) = make_float2(acc[nb][2], acc[nb][3]);
     }
     if (tid < H) {
-        part_ml[((size_t)s * H + tid) * 2 + 0] = mrun[tid];
-        part_ml[((size_t)s * H + tid) * 2 + 1] = lrun[tid];
+        part_ml[((size_t)s * d.heads + h0 + tid) * 2 + 0] = mrun[tid];
+        part_ml[((size_t)s * d.heads + h0 + tid) * 2 + 1] = lrun[tid];
     }
 }
 

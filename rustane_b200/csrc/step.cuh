@@ -133,9 +133,10 @@ cudaError_t launch_gemv(cd_model* m, const void* W, const float* x, const float*
 
 // What follows the layers: nothing (hidden state wanted), or the final RMSNorm + LM head and the head reduction /
 // sampler the step asks for.  `ars`: all-reduces the token issued (tensor / expert parallel), `last_ar`: index of the
-// one whose sum is still in the inboxes.  WT: storage of the LM head; LT: row format of the next token's first GEMV.
-template <typename WT, typename LT>
-cudaError_t enqueue_head_t(cd_model* m, const cd_step& p, bool use_mega, unsigned int ars, int last_ar) {
+// one whose sum is still in the inboxes.  WT: storage of the LM head; LT: row format of the next token's first GEMV; HeadIn:
+// how the head's input comes about where that is not RMSNorm of x_a (an input type of the streamed GEMV, kernels.cuh).
+template <typename WT, typename LT, class HeadIn = GemvIn>
+cudaError_t enqueue_head_t(cd_model* m, const cd_step& p, bool use_mega, unsigned int ars, int last_ar, const HeadIn& head_in = HeadIn{}) {
     const cd_config& c = m->cfg;
     cudaError_t e;
 #define TRY(x) do { e = (x); if (e != cudaSuccess) return e; } while (0)
@@ -160,7 +161,8 @@ cudaError_t enqueue_head_t(cd_model* m, const cd_step& p, bool use_mega, unsigne
     m->next_stream = NextStream{m->prefetch_kb > 0 ? m->layers[0].wqkv : nullptr, Wfmt<LT>::row_stride(c.dim),
                                 (c.q_dim + 2 * c.kv_dim) / 2, 2, (uint32_t)m->prefetch_kb * 1024u};
     if (m->tp_world > 1) { m->tp_in.in_reduce = last_ar; m->tp_in.res = m->x_b; m->tp_in.x_out = m->x_a; }
-    TRY((launch_gemv<WT, 1, true>(m, m->lm_head, m->x_a, m->gamma_final, m->norm_final, m->v_loc, c.dim, EpiStore{m->logits})));
+    if constexpr (HeadIn::CUSTOM) TRY((launch_gemv<WT, 1, false>(m, m->lm_head, m->x_a, nullptr, nullptr, m->v_loc, c.dim, EpiStore{m->logits}, SrcPlain{}, head_in)));
+    else TRY((launch_gemv<WT, 1, true>(m, m->lm_head, m->x_a, m->gamma_final, m->norm_final, m->v_loc, c.dim, EpiStore{m->logits})));
     }
     unsigned int* head_counter = m->counters + c.heads;
     m->cur_cls = CLS_SAMPLE;
