@@ -286,6 +286,57 @@ DAFIDRA_SIZES = {
 }
 
 
+def kazodra_config(width, heads, kv_heads, rank, window, ff, side, pattern, layers):
+    """A Kazodra configuration that repeats `pattern` (a: differential attention, l: latent attention, s: linear attention),
+    head widths as in the families it is compared with."""
+    mixers = {
+        "a": ("attention", {"heads": heads, "kv_heads": kv_heads, "dim": 64, "vdim": 128, "scale": 0.125, "diff": 0.5,
+                            "rot": {"dims": 64, "base": 500000.0, "scaling": {"factor": 8.0, "low": 1.0, "high": 4.0, "original": 2048}}}),
+        "l": ("latent_attention", {"heads": heads, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": rank, "scale": 192 ** -0.5,
+                                   "rot": {"dims": 64, "base": 10000.0}, "mask": {"size": window}}),
+        "s": ("lightning", {"heads": heads, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** -(2 + 8.0 * h / heads) for h in range(heads)]}),
+    }
+    out = [{"type": mixers[k][0], "mixer": mixers[k][1], "mlp": {"kind": "dense", "ff": ff}} for k in (pattern * layers)[:layers]]
+    cfg = {"architecture": "Kazodra", "width": width, "vocab": 32000, "norm": {"eps": 1e-5}, "layers": out}
+    if side:
+        cfg["token_side"] = {"dim": side}
+    return cfg
+
+
+# name -> (Kazodra configuration, the existing configured decoder or family it is compared with at equal width, depth and FFN columns)
+KAZODRA_SIZES = {
+    "1b": (kazodra_config(2048, 16, 4, 512, 1024, 5632, 128, "lssa", 24), "1b_dense"),
+    "5b": (kazodra_config(4096, 32, 8, 512, 1024, 11008, 128, "lssa", 26), "5b_dense"),
+    "1b_latent": (kazodra_config(2048, 16, 4, 512, 0x10000, 5632, 0, "l", 24), "moe_mla"),      # whole context visible, like its neighbour
+    "1b_linear": (kazodra_config(2048, 16, 4, 512, 1024, 5632, 0, "s", 24), "1b_dense"),
+    "1b_differential": (kazodra_config(2048, 16, 4, 512, 1024, 5632, 0, "a", 24), "dense"),
+}
+
+
+def kazodra_bytes(cfg, ctx):
+    """Algorithmic HBM bytes of one decoded token by kernel class (bf16 weights, fp16 cache, fp32 state read and written)."""
+    D, out = cfg["width"], dict.fromkeys(("qkv_gemv", "attention", "wo_gemv", "w13_gemv", "w2_gemv", "misc"), 0)
+    side = (cfg.get("token_side") or {}).get("dim", 0)
+    for L in cfg["layers"]:
+        c, H = L["mixer"], L["mixer"]["heads"]
+        if L["type"] == "latent_attention":
+            rows, w = H * (c["dim"] + c["rot_dim"]) + c["kv_rank"] + c["rot_dim"], c["kv_rank"] + c["rot_dim"]
+            out["attention"] += min(c["mask"]["size"], ctx) * w * 2 + c["kv_rank"] * H * (c["dim"] + c["vdim"]) * 2
+        elif L["type"] == "lightning":
+            rows = 2 * H * (c["dim"] + c["vdim"])
+            out["attention"] += 2 * 4 * H * c["dim"] * c["vdim"]
+        else:
+            rows = 2 * c["dim"] * (H + c["kv_heads"]) + c["vdim"] * (H + c["kv_heads"])
+            out["attention"] += ctx * c["kv_heads"] * (2 * c["dim"] + c["vdim"]) * 2
+        out["qkv_gemv"] += rows * D * 2
+        out["wo_gemv"] += D * H * c["vdim"] * 2
+        out["w13_gemv"] += 2 * L["mlp"]["ff"] * D * 2
+        out["w2_gemv"] += L["mlp"]["ff"] * D * 2
+        out["misc"] += 2 * side * D * 2
+    out["head_gemv"] = cfg["vocab"] * D * 2
+    return out
+
+
 def dafidra_bytes(cfg, ctx):
     """Algorithmic HBM bytes of one decoded token by kernel class (bf16 weights, fp16 cache, fp32 state read and written)."""
     D, out = cfg["width"], dict.fromkeys(("qkv_gemv", "attention", "wo_gemv", "w13_gemv", "w2_gemv"), 0)
@@ -320,8 +371,8 @@ def existing_bytes(kind, c, ctx):
     return out
 
 
-def bench_dafidra(sizes):
-    """Prefill and decode throughput of the Dafidra decoder (random weights) beside the closest existing family at equal
+def bench_configured(family, sizes):
+    """Prefill and decode throughput of a configured decoder (random weights) beside the closest existing family at equal
     size, with the time and roofline fraction of every kernel class of one token.  Prints one JSON line per size."""
     import numpy as np
 
@@ -356,34 +407,49 @@ def bench_dafidra(sizes):
         model.close()
         return out
 
+    prompts, measured = (1024, 2048, 4096), {}
+
+    def configured(cfg, by_class):
+        return measure(R.Model.from_config(cfg, 7, max_tokens=8192, use_graph=True), cfg["vocab"], by_class, prompts)
+
+    def existing(which):
+        if which in DAFIDRA_SIZES and family == "kazodra":
+            cfg = DAFIDRA_SIZES[which][0]
+            return "dafidra", lambda: configured(cfg, dafidra_bytes(cfg, ctx))
+        kind, dims = DAFIDRA_SIZES[which if which in DAFIDRA_SIZES else "moe" if which == "moe_mla" else "1b_dense"][1]
+        if kind == "dense":  # (four query heads per kv head: one kernel per operator, like the configured decoder)
+            return kind, lambda: measure(R.Model.synthetic(R.Config(**dims), 7, dtype="bf16", use_graph=True), dims["vocab"], existing_bytes(kind, dims, ctx), prompts)
+        return kind, lambda: measure(R.Model.moe_synthetic(R.MoeConfig(**dims), 7, dtype="bf16", use_graph=True), dims["vocab"], existing_bytes(kind, dims, ctx), ())
+
     for name in sizes:
-        cfg, (closest, dims) = DAFIDRA_SIZES[name]
+        cfg, which = (KAZODRA_SIZES if family == "kazodra" else DAFIDRA_SIZES)[name]
+        if family == "dafidra":
+            which = name
         line = {"size": name, "hbm_peak_gbs": peak, "peak_source": kind, "context": ctx, "decode_steps": steps,
                 "l2": "weights larger than L2 stream from HBM for every token and prompt pass", "data": "synthetic", "dtype": "bf16"}
         sampler = ClockSampler(0)
         sampler.start()
-        line["dafidra"] = measure(R.Model.from_config(cfg, 7, max_tokens=8192, use_graph=True), cfg["vocab"], dafidra_bytes(cfg, ctx), (1024, 2048, 4096))
-        if closest == "dense":  # (four query heads per kv head: one kernel per operator, like the configured decoder)
-            line[closest] = measure(R.Model.synthetic(R.Config(**dims), 7, dtype="bf16", use_graph=True), dims["vocab"], existing_bytes(closest, dims, ctx),
-                                    (1024, 2048, 4096))
-        else:
-            line[closest] = measure(R.Model.moe_synthetic(R.MoeConfig(**dims), 7, dtype="bf16", use_graph=True), dims["vocab"], existing_bytes(closest, dims, ctx), ())
+        line[family] = configured(cfg, (kazodra_bytes if family == "kazodra" else dafidra_bytes)(cfg, ctx))
+        closest, run = existing(which)
+        if which not in measured:
+            measured[which] = run()
+        line[closest] = measured[which]
         line["clocks"] = sampler.stop()
         print(json.dumps(line), flush=True)
 
 
-def profile_dafidra(size, prompt):
-    """Small case for `ncu` on the Dafidra decoder: two layers of one of the sizes; a prompt pass, then eight tokens."""
+def profile_configured(sizes, size, layers, prompt):
+    """Small case for `ncu` on a configured decoder: the first layers of one of the sizes; a prompt pass, then eight tokens."""
     import rustane_b200 as R
-    cfg = dict(DAFIDRA_SIZES[size][0])
-    cfg["layers"] = cfg["layers"][:2]
+    cfg = dict(sizes[size][0])
+    cfg["layers"] = cfg["layers"][:layers]
     model = R.Model.from_config(cfg, 7, max_tokens=8192)
     for _ in range(2):
         model.set_len(0)
         model.prefill(R.synth_prompt(3, cfg["vocab"], prompt))
     ms = model.last_device_ms()
     model.decode_steps_greedy(1, 8)
-    print("Dafidra profile case done: %d launches, prompt pass %.3f ms, %.3f ms/token" % (model.kernel_launches(), ms, model.last_device_ms() / 8))
+    print(cfg["architecture"] + " profile case done: %d launches, prompt pass %.3f ms, %.3f ms/token" % (model.kernel_launches(), ms, model.last_device_ms() / 8))
 
 
 def profile_case(dtype="bf16", per_operator=False):
@@ -462,11 +528,19 @@ def main():
                     help="prefill and decode throughput of the Dafidra decoder beside the closest existing family (all sizes, or the named ones)")
     ap.add_argument("--profile-dafidra", choices=sorted(DAFIDRA_SIZES), default=None,
                     help="small case for ncu captures of the Dafidra decoder (two layers of a size, a 2048-token prompt, 8 tokens); prints no bench line")
+    ap.add_argument("--kazodra", nargs="*", choices=sorted(KAZODRA_SIZES), default=None,
+                    help="prefill and decode throughput of the Kazodra decoder beside the closest existing family (all sizes, or the named ones)")
+    ap.add_argument("--profile-kazodra", choices=sorted(KAZODRA_SIZES), default=None,
+                    help="small case for ncu captures of the Kazodra decoder (four layers of a size, a 2048-token prompt, 8 tokens); prints no bench line")
     args = ap.parse_args()
     if args.dafidra is not None:
-        return bench_dafidra(args.dafidra or sorted(DAFIDRA_SIZES))
+        return bench_configured("dafidra", args.dafidra or sorted(DAFIDRA_SIZES))
     if args.profile_dafidra:
-        return profile_dafidra(args.profile_dafidra, 2048)
+        return profile_configured(DAFIDRA_SIZES, args.profile_dafidra, 2, 2048)
+    if args.kazodra is not None:
+        return bench_configured("kazodra", args.kazodra or sorted(KAZODRA_SIZES))
+    if args.profile_kazodra:
+        return profile_configured(KAZODRA_SIZES, args.profile_kazodra, 4, 2048)
     if args.profile_case:
         return profile_case(args.dtype, args.per_operator)
     if args.profile_moe:

@@ -150,7 +150,7 @@ cudaError_t hybrid_step_t(cd_model* m, const cd_step& p) {
         }
         if (f.kind != FfnCfg::NONE) behind = {S.y2, L.post2, nullptr};
         if (side) {
-            m->cur_cls = CLS_W2;
+            m->cur_cls = CLS_MISC;
             hint(L.side_proj, S.side_pad(), D, 1);
             const EpiTokenGate<WT> to_side{S.side, (const WT*)S.side_embed + (size_t)S.runs[r].layer * side, S.side_ld(), m->full_cfg.vocab, m->st};
             TRY((launch_gemv<WT, 1, false>(m, L.side_gate, x[cur], nullptr, nullptr, side, D, to_side, SrcPlain{}, residual(VecNorm{}))));

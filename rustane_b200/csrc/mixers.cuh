@@ -286,9 +286,11 @@ struct InGatedNorm {
 #pragma unroll
             for (int e = 0; e < EPC; e += 4) {
                 float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-                if (c < nchunks) v = __ldcg(reinterpret_cast<const float4*>(mem + (size_t)c * EPC + e));  // zeros behind the last head
+                if (c < nchunks) v = __ldcg(reinterpret_cast<const float4*>(mem + (size_t)c * EPC + e));
                 xr[i][e] = v.x; xr[i][e + 1] = v.y; xr[i][e + 2] = v.z; xr[i][e + 3] = v.w;
-                ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+#pragma unroll
+                for (int k = 0; k < 4; ++k)
+                    if (c * EPC + e + k < n) ss = fmaf(xr[i][e + k], xr[i][e + k], ss);  // another layer's values may lie behind the last head
             }
         }
         const float r = 1.0f / sqrtf(consumer_sum(ss, red, group) / (float)n + eps);
