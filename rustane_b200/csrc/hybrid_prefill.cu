@@ -183,7 +183,8 @@ int run_piece(cd_model* m, HybridPrefill* w, float* x, const uint32_t* ids, int 
         const float *add_ffn = side ? nullptr : next_add, *add_mixer = f.kind != FfnCfg::NONE ? nullptr : add_ffn;
         const ProjLayout& pl = L.proj;
         const int proj_ld = (int)round_up(pl.rows, 32);
-        gemm("projections", xn, xn_lo, L.wmix, rows, pl.rows, D, pl.rows, PfEpiPartial{w->proj, proj_ld});
+        const int activated = L.md.linear() ? pl.rg : 0;  // q, k and v of a linear attention
+        gemm("projections", xn, xn_lo, L.wmix, rows, pl.rows, D, pl.rows, PfEpiPartial{w->proj, proj_ld, activated});
         KT* q = (KT*)w->q;
         KT* pool = (KT*)m->layers[r].kv;
         AT* attn = w->attn;

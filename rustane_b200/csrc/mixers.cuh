@@ -515,7 +515,7 @@ __device__ inline void attn_step(const MixerStep& p, KT* __restrict__ pool, int 
         auto entry = [&](const float* src, const float* norm, int head, int i, float r) {
             const int q = i / a.kp, d = i % a.kp, at = (head * MAPS + q) * a.dim;
             if (d >= a.dim) return 0.0f;
-            return a.rot.entry(pos, d, [&](int j) { return __ldcg(src + at + j) * r * (norm != nullptr ? norm[at + j] : 1.0f); });
+            return a.rot.entry(d, [&](int k) { return a.rot.at(pos, k); }, [&](int j) { return __ldcg(src + at + j) * r * (norm != nullptr ? norm[at + j] : 1.0f); });
         };
         for (int i = tid; i < kr; i += MIX_THREADS) qs[i] = entry(p.proj + p.pl.lq, p.q_norm, h, i, rq);
         if (newest) {
@@ -696,8 +696,14 @@ __device__ inline void attn_step(const MixerStep& p, KT* __restrict__ pool, int 
         for (int q = 0; q < MAPS; ++q) {
             const float* pa = p.part_acc + (size_t)(h * MAPS + q) * p.nsplit * a.vp + i;
             float o = 0.0f;
-#pragma unroll 4
-            for (int s = 0; s < used; ++s) o = fmaf(__ldcg(pa + (size_t)s * a.vp), ps[q * MIX_TILE + s], o);
+            for (int s0 = 0; s0 < used; s0 += 16) {  // sixteen slices in flight together
+                float t[16];
+#pragma unroll
+                for (int s = 0; s < 16; ++s) t[s] = s0 + s < used ? __ldcg(pa + (size_t)(s0 + s) * a.vp) : 0.0f;
+#pragma unroll
+                for (int s = 0; s < 16; ++s)
+                    if (s0 + s < used) o = fmaf(t[s], ps[q * MIX_TILE + s0 + s], o);
+            }
             r = fmaf(o, inv[q], r);
         }
         vc[i] = r;  // each thread reads its own entries again

@@ -36,6 +36,9 @@ __global__ void __launch_bounds__(256) attn_rows_kernel(const float* __restrict_
         rq /= sqrtf(block_sum(sq, red) / (float)nq + a.eps);
         rk = 1.0f / sqrtf(block_sum(sk, red) / (float)nk + a.eps);
     }
+    __shared__ float2 cs_sm[128];  // dims is at most 256
+    a.rot.fill(cs_sm, pos);
+    __syncthreads();
     // two neighbouring entries (a rotated pair) of a [head][map][kp] vector
     auto pair = [&](const float* src, const float* norm, int i, float r, float& u, float& v) {
         const int hm = i / a.kp, d = i % a.kp;
@@ -43,7 +46,7 @@ __global__ void __launch_bounds__(256) attn_rows_kernel(const float* __restrict_
         u = d < a.dim ? p[d] * r * (norm != nullptr ? norm[hm * a.dim + d] : 1.0f) : 0.0f;
         v = d + 1 < a.dim ? p[d + 1] * r * (norm != nullptr ? norm[hm * a.dim + d + 1] : 1.0f) : 0.0f;
         if (d < a.rot.dims) {
-            const float2 cs = a.rot.at(pos, d >> 1);
+            const float2 cs = cs_sm[d >> 1];
             const float t = u * cs.x - v * cs.y;
             v = v * cs.x + u * cs.y;
             u = t;
@@ -293,10 +296,14 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const float* __restric
     __shared__ float red[32];
     const float* row = proj + (size_t)blockIdx.x * ld;
     const int pos = pos0 + blockIdx.x, tid = threadIdx.x, QH = d.nope_n + d.rope_n;
+    __shared__ float2 cs_sm[128];  // nope + rope is at most 256
+    auto cs_of = [&](int k) { return cs_sm[k]; };
+    rot.fill(cs_sm, pos);
+    __syncthreads();
     for (int i = tid; i < d.heads * kp; i += 256) {
         const int h = i / kp, k = i % kp;
         const float* q = row + h * QH;
-        const float v = k < d.nope_n ? q[k] : k < QH ? rot.entry(pos, k - d.nope_n, [&](int j) { return q[d.nope_n + j]; }) : 0.0f;
+        const float v = k < d.nope_n ? q[k] : k < QH ? rot.entry(k - d.nope_n, cs_of, [&](int j) { return q[d.nope_n + j]; }) : 0.0f;
         pf_store(q_hi, q_lo, (size_t)blockIdx.x * d.heads * kp + i, v);
     }
     const float* craw = row + d.heads * QH;
@@ -305,7 +312,7 @@ __global__ void __launch_bounds__(256) latent_rows_kernel(const float* __restric
     const float r = 1.0f / sqrtf(block_sum(ss, red) / (float)d.latent_n + d.eps);
     KT* out = pool + ((size_t)page_table[pos / d.page_tokens] * d.page_tokens + pos % d.page_tokens) * d.row();
     for (int i = tid; i < d.latent; i += 256) out[i] = Elem<KT>::from_f32(i < d.latent_n ? craw[i] * r * gamma[i] : 0.0f);
-    for (int i = tid; i < d.rope; i += 256) out[d.latent + i] = Elem<KT>::from_f32(i < d.rope_n ? rot.entry(pos, i, [&](int j) { return craw[d.latent_n + j]; }) : 0.0f);
+    for (int i = tid; i < d.rope; i += 256) out[d.latent + i] = Elem<KT>::from_f32(i < d.rope_n ? rot.entry(i, cs_of, [&](int j) { return craw[d.latent_n + j]; }) : 0.0f);
 }
 
 // cached rows base, base + 1, ..: the latent as a GEMM operand [n][latent], the rotated key behind every head's expanded one
@@ -336,6 +343,13 @@ template <typename KT> struct PfEpiExpand {
         bool key = col < keys;
         if (h >= x.H) return;
         KT* dst = expanded + (key ? x.k_at(0, h, row) : x.v_at(0, h, row));
+        if (nope % 32 == 0 && x.vdim % 32 == 0) {  // the 32 columns are one head's, and so aligned
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+                *reinterpret_cast<uint4*>(dst + d + 8 * i) = make_uint4(pack2<KT>(v[8 * i], v[8 * i + 1]), pack2<KT>(v[8 * i + 2], v[8 * i + 3]),
+                                                                        pack2<KT>(v[8 * i + 4], v[8 * i + 5]), pack2<KT>(v[8 * i + 6], v[8 * i + 7]));
+            return;
+        }
 #pragma unroll
         for (int i = 0; i < 32; ++i) {
             dst[d] = Elem<KT>::from_f32(v[i]);
@@ -361,11 +375,14 @@ template <typename AT, typename WT> struct PfEpiTokenGate {
     const uint32_t* ids;
     __device__ void operator()(int, int row, int col, const float (&v)[32]) const {
         const WT* e = table + (size_t)ids[row] * table_ld;
+        float g[32];  // every entry is requested before anything is stored
 #pragma unroll
-        for (int i = 0; i < 32; ++i) {
-            const int c = col + i;
-            if (c < ld) pf_store(hi, lo, (size_t)row * ld + c, c < dim ? gelu_tanh(v[i]) * Elem<WT>::to_f32(e[c]) : 0.0f);
-        }
+        for (int i = 0; i < 32; ++i) g[i] = col + i < dim ? Elem<WT>::to_f32(__ldg(e + col + i)) : 0.0f;
+#pragma unroll
+        for (int i = 0; i < 32; ++i) g[i] *= gelu_tanh(v[i]);
+#pragma unroll
+        for (int i = 0; i < 32; ++i)
+            if (col + i < ld) pf_store(hi, lo, (size_t)row * ld + col + i, g[i]);
     }
 };
 
@@ -376,7 +393,7 @@ template <typename AT, typename WT> struct PfEpiTokenGate {
 // so a chunk needs only the state it starts from.  Three kernels: every chunk's own contribution to the state, a scan over
 // the chunks that turns the contributions into starting states, and the read-outs of all chunks.
 // Linear attention is the case with log forget gate ln(decay), input gate 1 and no maximum or normaliser: F_t = (t + 1) ln
-// decay, every scale e^0, and M_t = -F_t in the read-out.
+// decay, every scale e^0, and M_t = -F_t in the read-out; its q, k and v arrive activated.
 struct MemPrompt {
     MemDims d;
     ProjLayout pl;
@@ -425,16 +442,13 @@ __device__ inline void mem_chunk_gates(const MemPrompt& p, int h, int t0, int nt
     __syncthreads();
 }
 
-// a [64][64] tile of fp32 rows (act: through silu) as bf16 head and remainder; rows >= nrows and columns >= ncols are zero; row_scale may be null
-__device__ inline void mem_load_tile(__nv_bfloat16* hi, __nv_bfloat16* lo, const float* src, size_t ld, int nrows, int ncols, const float* row_scale, float scale, bool act = false) {
+// a [64][64] tile of fp32 rows as bf16 head and remainder; rows >= nrows and columns >= ncols are zero; row_scale may be null
+__device__ inline void mem_load_tile(__nv_bfloat16* hi, __nv_bfloat16* lo, const float* src, size_t ld, int nrows, int ncols, const float* row_scale, float scale) {
 #pragma unroll 8
     for (int i = threadIdx.x; i < 64 * 64; i += 128) {
         const int r = i >> 6, c = i & 63;
         float v = 0.0f;
-        if (r < nrows && c < ncols) {
-            v = src[(size_t)r * ld + c];
-            v = (act ? silu(v) : v) * (row_scale ? row_scale[r] : scale);
-        }
+        if (r < nrows && c < ncols) v = src[(size_t)r * ld + c] * (row_scale ? row_scale[r] : scale);
         pf_store(hi, lo, (size_t)r * MEM_LD + c, v);
     }
 }
@@ -487,8 +501,8 @@ static __global__ void __launch_bounds__(128) mem_chunk_kernel(const __grid_cons
     __syncthreads();
     __nv_bfloat16 *kh = tiles, *kl = tiles + MEM_TILE_ELEMS, *vh = tiles + 2 * MEM_TILE_ELEMS, *vl = tiles + 3 * MEM_TILE_ELEMS;
     const float* row0 = p.proj + (size_t)t0 * p.proj_ld;
-    mem_load_tile(kh, kl, row0 + p.pl.rk + h * d.dim + kb * 64, p.proj_ld, nt, d.dim - kb * 64, W, 1.0f, linear);
-    mem_load_tile(vh, vl, row0 + p.pl.rv + h * d.vdim + vb * 64, p.proj_ld, nt, d.vdim - vb * 64, nullptr, 1.0f, linear);
+    mem_load_tile(kh, kl, row0 + p.pl.rk + h * d.dim + kb * 64, p.proj_ld, nt, d.dim - kb * 64, W, 1.0f);
+    mem_load_tile(vh, vl, row0 + p.pl.rv + h * d.vdim + vb * 64, p.proj_ld, nt, d.vdim - vb * 64, nullptr, 1.0f);
     __syncthreads();
     float acc[8][4];
 #pragma unroll
@@ -606,7 +620,7 @@ static __global__ void __launch_bounds__(128) mem_out_kernel(const __grid_consta
     const float* S0 = p.U + ((size_t)c * d.H + h) * d.dim * d.vs;
     const float* N0 = p.UN + ((size_t)c * d.H + h) * d.dim;
     const float qscale = linear ? 1.0f : 1.0f / sqrtf((float)d.dim);
-    mem_load_tile(vh, vl, row0 + p.pl.rv + h * d.vdim + vb * 64, p.proj_ld, nt, d.vdim - vb * 64, nullptr, 1.0f, linear);
+    mem_load_tile(vh, vl, row0 + p.pl.rv + h * d.vdim + vb * 64, p.proj_ld, nt, d.vdim - vb * 64, nullptr, 1.0f);
     float sc[8][4], o[8][4], nq = 0.0f;
 #pragma unroll
     for (int i = 0; i < 8; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
@@ -614,8 +628,8 @@ static __global__ void __launch_bounds__(128) mem_out_kernel(const __grid_consta
     const uint32_t b_off = (uint32_t)((lane & 7) + 8 * (lane >> 4)) * (MEM_LD * 2) + (uint32_t)((lane >> 3) & 1) * 16u;
     for (int kb = 0; kb * 64 < d.dim; ++kb) {
         __syncthreads();  // the previous block's tiles are no longer read
-        mem_load_tile(qh, ql, row0 + p.pl.rq + h * d.dim + kb * 64, p.proj_ld, nt, d.dim - kb * 64, nullptr, qscale, linear);
-        mem_load_tile(kh, kl, row0 + p.pl.rk + h * d.dim + kb * 64, p.proj_ld, nt, d.dim - kb * 64, nullptr, 1.0f, linear);
+        mem_load_tile(qh, ql, row0 + p.pl.rq + h * d.dim + kb * 64, p.proj_ld, nt, d.dim - kb * 64, nullptr, qscale);
+        mem_load_tile(kh, kl, row0 + p.pl.rk + h * d.dim + kb * 64, p.proj_ld, nt, d.dim - kb * 64, nullptr, 1.0f);
         mem_load_tile(sh, sl, S0 + (size_t)kb * 64 * d.vs + vb * 64, d.vs, d.dim - kb * 64, d.vdim - vb * 64, nullptr, 1.0f);
         __syncthreads();
         if (!linear) {   // n_0 . q: two threads per token

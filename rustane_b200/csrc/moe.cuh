@@ -112,10 +112,14 @@ struct Rotation {
         sincosf(a, &cs.y, &cs.x);
         return cs;
     }
-    // entry d of a vector whose raw entries get(i) returns
-    template <class Get> __device__ float entry(int pos, int d, Get get) const {
+    // all of a position's rotations into shared memory (whole CTA; the caller's barrier publishes them)
+    __device__ void fill(float2* cs, int pos) const {
+        for (int k = threadIdx.x; k < dims / 2; k += blockDim.x) cs[k] = at(pos, k);
+    }
+    // entry d of a vector whose raw entries get(i) returns; cs(k) is the k-th rotation
+    template <class Cs, class Get> __device__ float entry(int d, Cs cs_of, Get get) const {
         if (d >= dims) return get(d);
-        const float2 cs = at(pos, d >> 1);
+        const float2 cs = cs_of(d >> 1);
         const float u = get(d & ~1), v = get(d | 1);
         return (d & 1) ? v * cs.x + u * cs.y : u * cs.x - v * cs.y;
     }
@@ -193,10 +197,15 @@ mla_post_kernel(const float* __restrict__ qa, const WT* __restrict__ wuk_t, cons
     pdl_wait();
     pdl_launch_dependents();
     const int pos = __ldcg(&st->pos);
+    float2* cs = reinterpret_cast<float2*>(sm + ((C + 1) & ~1));  // [dims / 2]
+    auto cs_of = [&](int k) { return cs[k]; };
+    rot.fill(cs, pos);
+    __syncthreads();
+#pragma unroll 4
     for (int i = tid; i < H * R; i += blockDim.x) {  // rotation of q's part of it
         const int h = i / R, k = i % R;
         const float* q = qa + (size_t)h * QH + d.nope_n;
-        put(h, C + k, k < d.rope_n ? rot.entry(pos, k, [&](int j) { return __ldcg(q + j); }) : 0.0f);
+        put(h, C + k, k < d.rope_n ? rot.entry(k, cs_of, [&](int j) { return __ldcg(q + j); }) : 0.0f);
     }
     // the cache row: normed latent | rotated key
     const float* craw = qa + (size_t)H * QH;
@@ -212,9 +221,9 @@ mla_post_kernel(const float* __restrict__ qa, const WT* __restrict__ wuk_t, cons
     KT* row = lat_pool + ((size_t)page * d.page_tokens + off) * (C + R);
     for (int i = tid; i < C; i += blockDim.x) row[i] = Elem<KT>::from_f32(i < d.latent_n ? sm[i] * inv * gamma_kv[i] : 0.0f);
     for (int i = tid; i < R; i += blockDim.x)
-        row[C + i] = Elem<KT>::from_f32(i < d.rope_n ? rot.entry(pos, i, [&](int j) { return __ldcg(craw + d.latent_n + j); }) : 0.0f);
+        row[C + i] = Elem<KT>::from_f32(i < d.rope_n ? rot.entry(i, cs_of, [&](int j) { return __ldcg(craw + d.latent_n + j); }) : 0.0f);
 }
-__host__ __device__ inline size_t mla_post_smem_floats(const MlaDims& d) { return max((128 / d.latent + 2) * d.nope, d.latent); }
+__host__ __device__ inline size_t mla_post_smem_floats(const MlaDims& d) { return max((128 / d.latent + 2) * d.nope, d.latent + 2 + d.rope); }
 
 // ---------------------------------------------------------------------- latent attention, one slice of cached positions per CTA
 // score_h(t) = qabs_h . row(t) * scale over the C + R wide cache row; out_h = sum_t p_h(t) row(t)[0 .. C).

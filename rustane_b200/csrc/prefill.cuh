@@ -116,11 +116,17 @@ template <typename T16> __device__ inline T16 pf_cast(float v);
 template <> __device__ inline __nv_bfloat16 pf_cast<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
 template <> __device__ inline __half pf_cast<__half>(float v) { return __float2half_rn(v); }
 
-struct PfEpiPartial {  // tensor parallel: this rank's partial product y, raw, for the all-reduce that follows
+struct PfEpiPartial {  // the product y, raw (tensor parallel: this rank's partial one, for the all-reduce that follows)
     float* y;
     int ld;
+    int silu_cols = 0;  // the first columns go through silu
     __device__ void operator()(int, int row, int col, const float (&v)[32]) const {
         float4* p = reinterpret_cast<float4*>(y + (size_t)row * ld + col);
+        if (col < silu_cols) {
+#pragma unroll
+            for (int i = 0; i < 32; ++i) reinterpret_cast<float*>(p)[i] = col + i < silu_cols ? v[i] / (1.0f + expf(-v[i])) : v[i];
+            return;
+        }
 #pragma unroll
         for (int i = 0; i < 8; ++i) p[i] = make_float4(v[4 * i], v[4 * i + 1], v[4 * i + 2], v[4 * i + 3]);
     }
