@@ -31,7 +31,7 @@ cudaError_t launch_mla(cd_model* m, const MlaStep& p) {
     cudaError_t e;
 #define TRY(x) do { e = (x); if (e != cudaSuccess) return e; } while (0)
     const bool mma = mla_on_tensor_cores<KT>(d);
-    TRY(launch_chain(m, mla_post_kernel<WT, KT>, dim3((d.heads * d.latent + 127) / 128 + 1), dim3(128), mla_post_smem_floats(d) * sizeof(float), p.qa, (const WT*)p.wuk_t,
+    TRY(launch_chain(m, mla_post_kernel<WT, KT>, dim3(mla_post_ctas(d)), dim3(128), mla_post_smem_floats(d) * sizeof(float), p.qa, (const WT*)p.wuk_t,
                      p.gamma, p.rot, (const int*)m->page_table, (const DevState*)m->st, (KT*)p.pool, p.qabs, mma ? (KT*)p.qsplit : (KT*)nullptr, d));
     if constexpr (!std::is_same<KT, float>::value) {
         if (mma) {

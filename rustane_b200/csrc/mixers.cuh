@@ -353,7 +353,7 @@ struct MixerStep {
     int nsplit;
 };
 constexpr int MIX_THREADS = 128, MIX_TILE = 32;
-__host__ __device__ inline size_t mixer_attn_smem_floats(int kr, int vp, int maps) { return (size_t)2 * kr + vp + (size_t)MIX_THREADS * 8 + (1 + maps) * MIX_TILE + 96; }
+__host__ __device__ inline size_t mixer_attn_smem_floats(int kr, int vp, int maps) { return (size_t)2 * kr + vp + (size_t)MIX_THREADS * 8 + (4 + maps) * MIX_TILE + 96; }
 __host__ __device__ inline size_t mixer_mem_smem_floats(int dim) { return (size_t)2 * dim + 4 * MEM_SLICE + 64; }
 
 // this thread's share of the sum of squares of n floats another kernel wrote
@@ -477,12 +477,13 @@ __device__ inline void attn_step(const MixerStep& p, KT* __restrict__ pool, int 
     const AttnDims& a = p.a;
     const int h = idx / p.nsplit, sl = idx % p.nsplit, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int gqa = a.H / a.G, g = h / gqa, kr = MAPS * a.kp;
-    float* qs = sm;                       // [MAPS][kp] query as it meets the keys: norm, rotation, temperature and scale folded in
+    size_t* k_off = reinterpret_cast<size_t*>(sm);  // [MIX_TILE] where the key and value rows of the tile's positions are
+    size_t* v_off = k_off + MIX_TILE;
+    float* qs = sm + 4 * MIX_TILE;        // [MAPS][kp] query as it meets the keys: norm, rotation, temperature and scale folded in
     float* kc = qs + kr;                  // [MAPS][kp] this position's key as the cache holds it
     float* vc = kc + kr;                  // [vp]
     float* accs = vc + a.vp;              // [128 threads][8]
     float* ps = accs + MIX_THREADS * 8;   // [MAPS][MIX_TILE]
-    int* pages = reinterpret_cast<int*>(ps + MAPS * MIX_TILE);  // [MIX_TILE] page of each position of the tile
     pdl_wait();
     pdl_launch_dependents();
     const int pos = __ldcg(&p.st->pos);
@@ -504,7 +505,14 @@ __device__ inline void attn_step(const MixerStep& p, KT* __restrict__ pool, int 
     const int vch = tid % lv, vgrp = tid / lv, vgroups = MIX_THREADS / lv;
     if (t0 < t1) {
         const bool newest = t1 == pos + 1;  // this slice holds the current position
-        if (tid < MIX_TILE) pages[tid] = p.page_table[min(t0 + tid, pos) / a.page_tokens];
+        auto locate = [&](int tb) {
+            if (tid < MIX_TILE) {
+                const int t = min(tb + tid, pos), page = p.page_table[t / a.page_tokens], off = t % a.page_tokens;
+                k_off[tid] = a.k_at(page, g, off);
+                v_off[tid] = a.v_at(page, g, off);
+            }
+        };
+        locate(t0);
         float rq = a.temperature(pos) * a.scale, rk = 1.0f;
         if (p.q_norm != nullptr) {
             const float sq = sum_of_squares(p.proj + p.pl.lq, a.H * MAPS * a.dim), sk = newest ? sum_of_squares(p.proj + p.pl.lk, a.G * MAPS * a.dim) : 0.0f;
@@ -547,7 +555,7 @@ __device__ inline void attn_step(const MixerStep& p, KT* __restrict__ pool, int 
             for (int u = 0; u < PRE; ++u) {
                 const int j = vgrp + u * vgroups;
                 vw[u] = make_uint4(0, 0, 0, 0);
-                if (vch < nvc && j < nt && tb + j != pos) vw[u] = ldg_stream_coherent(pool + a.v_at(pages[j], g, (tb + j) % a.page_tokens) + (size_t)vch * EPC);
+                if (vch < nvc && j < nt && tb + j != pos) vw[u] = ldg_stream_coherent(pool + v_off[j] + (size_t)vch * EPC);
             }
             // scores: warp w takes positions tb + 8 w .. + 7
             for (int j0 = 0; j0 < 8; j0 += 4 * side) {
@@ -562,7 +570,7 @@ __device__ inline void attn_step(const MixerStep& p, KT* __restrict__ pool, int 
                     for (int u = 0; u < 4; ++u) {
                         const int j = j0 + u * side + lane / lk, t = tb + 8 * warp + j;
                         const bool cached = j < 8 && t < t1 && t != pos;
-                        const KT* row = pool + (cached ? a.k_at(pages[8 * warp + j], g, t % a.page_tokens) : 0) + (size_t)c * EPC;
+                        const KT* row = pool + (cached ? k_off[8 * warp + j] : 0) + (size_t)c * EPC;
 #pragma unroll
                         for (int q = 0; q < MAPS; ++q) w[u][q] = cached ? ldg_stream_coherent(row + (size_t)q * a.kp) : make_uint4(0, 0, 0, 0);
                     }
@@ -635,11 +643,11 @@ __device__ inline void attn_step(const MixerStep& p, KT* __restrict__ pool, int 
                     if (vgrp + u * vgroups < nt) add(vgrp + u * vgroups, vw[u]);
 #pragma unroll 4
                 for (int j = vgrp + PRE * vgroups; j < nt; j += vgroups)
-                    add(j, tb + j == pos ? make_uint4(0, 0, 0, 0) : ldg_stream_coherent(pool + a.v_at(pages[j], g, (tb + j) % a.page_tokens) + (size_t)vch * EPC));
+                    add(j, tb + j == pos ? make_uint4(0, 0, 0, 0) : ldg_stream_coherent(pool + v_off[j] + (size_t)vch * EPC));
             }
-            __syncthreads();  // the tile's pages and probabilities are no longer read
+            __syncthreads();  // the tile's places and probabilities are no longer read
             if (tb + MIX_TILE < t1) {
-                if (tid < MIX_TILE) pages[tid] = p.page_table[min(tb + MIX_TILE + tid, pos) / a.page_tokens];
+                locate(tb + MIX_TILE);
                 __syncthreads();
             }
         }

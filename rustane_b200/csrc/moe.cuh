@@ -126,10 +126,10 @@ struct Rotation {
 };
 
 // ---------------------------------------------------------------------- after the q | latent | key GEMV
-// grid = ceil(heads * C / 128) + 1 CTAs of 128 threads.  The first CTAs: one thread per row (h, c) of the absorbed-key matrix,
-// q'_h[c] = sum_d W_uk[c, h N + d] q_nope_h[d] (a row is N elements: every thread has its whole row in flight);
-// the last CTA: RoPE on the heads' RoPE parts of q, and the cache row of this position
-// [rmsnorm(latent) | rope(key)].  qabs[h] = [q'_h (C) | rope(q_rope_h) (R)].
+// CTAs of 128 threads.  The first ceil(heads * C / 128): one thread per row (h, c) of the absorbed-key matrix,
+// q'_h[c] = sum_d W_uk[c, h N + d] q_nope_h[d] (a row is N elements: every thread has its whole row in flight); the next
+// ceil(heads * R / 256): RoPE on the heads' RoPE parts of q, a pair per thread; the last CTA: the cache row of this
+// position [rmsnorm(latent) | rope(key)].  qabs[h] = [q'_h (C) | rope(q_rope_h) (R)].
 template <typename WT, typename KT>
 __global__ void __launch_bounds__(128)
 mla_post_kernel(const float* __restrict__ qa, const WT* __restrict__ wuk_t, const float* __restrict__ gamma_kv, Rotation rot,
@@ -151,7 +151,8 @@ mla_post_kernel(const float* __restrict__ qa, const WT* __restrict__ wuk_t, cons
             q[(size_t)16 * (C + R)] = Elem<KT>::from_f32(v - Elem<KT>::to_f32(hi));
         }
     };
-    if (blockIdx.x + 1 < gridDim.x) {
+    const int n_absorb = (H * C + 127) / 128;
+    if ((int)blockIdx.x < n_absorb) {
         const int r = min((int)(blockIdx.x * blockDim.x) + tid, H * C - 1);  // row (h, c)
         const char* row = reinterpret_cast<const char*>(wuk_t + (size_t)r * N);
         constexpr int PRE = 16;  // chunks of the row requested before anything else (a whole 128-wide 16-bit row)
@@ -197,24 +198,33 @@ mla_post_kernel(const float* __restrict__ qa, const WT* __restrict__ wuk_t, cons
     pdl_wait();
     pdl_launch_dependents();
     const int pos = __ldcg(&st->pos);
-    float2* cs = reinterpret_cast<float2*>(sm + ((C + 1) & ~1));  // [dims / 2]
-    auto cs_of = [&](int k) { return cs[k]; };
-    rot.fill(cs, pos);
-    __syncthreads();
-#pragma unroll 4
-    for (int i = tid; i < H * R; i += blockDim.x) {  // rotation of q's part of it
-        const int h = i / R, k = i % R;
+    if (blockIdx.x + 1 < gridDim.x) {  // rotation of q's part of it
+        const int i = 2 * (((int)blockIdx.x - n_absorb) * (int)blockDim.x + tid), h = i / R, k = i % R;
+        if (i >= H * R) return;
         const float* q = qa + (size_t)h * QH + d.nope_n;
-        put(h, C + k, k < d.rope_n ? rot.entry(k, cs_of, [&](int j) { return __ldcg(q + j); }) : 0.0f);
+        float u = k < d.rope_n ? __ldcg(q + k) : 0.0f, v = k + 1 < d.rope_n ? __ldcg(q + k + 1) : 0.0f;
+        if (k < rot.dims) {
+            const float2 cs = rot.at(pos, k >> 1);
+            const float t = u * cs.x - v * cs.y;
+            v = v * cs.x + u * cs.y;
+            u = t;
+        }
+        put(h, C + k, u);
+        put(h, C + k + 1, v);
+        return;
     }
     // the cache row: normed latent | rotated key
     const float* craw = qa + (size_t)H * QH;
+    float2* cs = reinterpret_cast<float2*>(sm + ((C + 1) & ~1));  // [dims / 2]
+    auto cs_of = [&](int k) { return cs[k]; };
     float ss = 0.0f;
+#pragma unroll 8
     for (int i = tid; i < d.latent_n; i += blockDim.x) {
         const float v = __ldcg(craw + i);
         sm[i] = v;
         ss += v * v;
     }
+    rot.fill(cs, pos);
     const float tot = block_sum(ss, red);
     const float inv = 1.0f / sqrtf(tot * (1.0f / (float)d.latent_n) + d.eps);
     const int page = page_table[pos / d.page_tokens], off = pos % d.page_tokens;
@@ -224,6 +234,7 @@ mla_post_kernel(const float* __restrict__ qa, const WT* __restrict__ wuk_t, cons
         row[C + i] = Elem<KT>::from_f32(i < d.rope_n ? rot.entry(i, cs_of, [&](int j) { return __ldcg(craw + d.latent_n + j); }) : 0.0f);
 }
 __host__ __device__ inline size_t mla_post_smem_floats(const MlaDims& d) { return max((128 / d.latent + 2) * d.nope, d.latent + 2 + d.rope); }
+__host__ __device__ inline int mla_post_ctas(const MlaDims& d) { return (d.heads * d.latent + 127) / 128 + (d.heads * d.rope + 255) / 256 + 1; }
 
 // ---------------------------------------------------------------------- latent attention, one slice of cached positions per CTA
 // score_h(t) = qabs_h . row(t) * scale over the C + R wide cache row; out_h = sum_t p_h(t) row(t)[0 .. C).
