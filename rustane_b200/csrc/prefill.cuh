@@ -124,7 +124,7 @@ struct PfEpiPartial {  // the product y, raw (tensor parallel: this rank's parti
         float4* p = reinterpret_cast<float4*>(y + (size_t)row * ld + col);
         if (col < silu_cols) {
 #pragma unroll
-            for (int i = 0; i < 32; ++i) reinterpret_cast<float*>(p)[i] = col + i < silu_cols ? v[i] / (1.0f + expf(-v[i])) : v[i];
+            for (int i = 0; i < 32; ++i) reinterpret_cast<float*>(p)[i] = col + i < silu_cols ? __fdividef(v[i], 1.0f + __expf(-v[i])) : v[i];
             return;
         }
 #pragma unroll

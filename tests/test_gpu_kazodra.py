@@ -239,6 +239,22 @@ def test_wide_rows(R, tmp_path):
             assert M.error(all_logits(m, ids), ref) < 2 * TOL[dtype]
 
 
+@pytest.mark.parametrize("dtype", ["f32", "bf16"])
+@pytest.mark.parametrize("width,side", [(64, 1), (200, 9), (1024, 300), (1024, 700)])
+def test_token_side_sizes(R, tmp_path, width, side, dtype):
+    """From one column per layer to widths of several GEMM tiles, at and off multiples of 8."""
+    cfg = M.config(width, 90, [(M.lightning(2, 8, 12, (0.5, 0.9)), None), (M.latent(2, 8, 4, 8, 16, 9, 0.3), 24)], side=side)
+    W = M.weights(cfg, 4)
+    ids = np.random.default_rng(6).integers(0, 90, 40)
+    ref = K.forward(cfg, M.f64(W), ids)
+    assert M.error(K.forward(cfg, M.f64(W), ids, fault="first_part"), ref) > 0.1
+    m = R.Model.from_pretrained(folder(tmp_path, cfg, W), max_tokens=40, dtype=dtype, use_graph=True)
+    one = np.stack([m.decode_token_logits_from_id(int(t)) for t in ids])
+    assert M.error(one, ref) < TOL[dtype]
+    m.set_len(0)
+    assert M.error(all_logits(m, ids, [30, 10]), ref) < TOL[dtype]
+
+
 # ---------------------------------------------------------------------- sequences one after the other, rewinding
 def test_cache_and_state_are_clean_for_the_next_sequence(R, made):
     cfg, _, path, ids, ref = made("ODD")
