@@ -375,14 +375,29 @@ template <typename AT, typename WT> struct PfEpiTokenGate {
     const uint32_t* ids;
     __device__ void operator()(int, int row, int col, const float (&v)[32]) const {
         const WT* e = table + (size_t)ids[row] * table_ld;
-        float g[32];  // every entry is requested before anything is stored
+        float g[32];
+        const bool run = col + 32 <= dim && table_ld % 8 == 0 && (reinterpret_cast<size_t>(table) & 15) == 0;
+        if (run) {
 #pragma unroll
-        for (int i = 0; i < 32; ++i) g[i] = col + i < dim ? Elem<WT>::to_f32(__ldg(e + col + i)) : 0.0f;
+            for (int i = 0; i < 32; i += 8) {
+                float f[8];
+                Elem<WT>::unpack(ldg_stream(e + col + i), f);
+#pragma unroll
+                for (int k = 0; k < 8; ++k) g[i + k] = f[k];
+            }
+        } else {  // every entry is requested before anything is stored
+#pragma unroll
+            for (int i = 0; i < 32; ++i) g[i] = col + i < dim ? Elem<WT>::to_f32(__ldg(e + col + i)) : 0.0f;
+        }
 #pragma unroll
         for (int i = 0; i < 32; ++i) g[i] *= gelu_tanh(v[i]);
+        if (run) {  // (dim >= col + 32, so the operand's rows hold them)
+            pf_store_run(hi, lo, (size_t)row * ld + col, g);
+        } else {
 #pragma unroll
-        for (int i = 0; i < 32; ++i)
-            if (col + i < ld) pf_store(hi, lo, (size_t)row * ld + col + i, g[i]);
+            for (int i = 0; i < 32; ++i)
+                if (col + i < ld) pf_store(hi, lo, (size_t)row * ld + col + i, g[i]);
+        }
     }
 };
 

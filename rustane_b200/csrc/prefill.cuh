@@ -154,12 +154,30 @@ template <typename T16> __device__ inline void pf_store(T16* hi, T16* lo, size_t
     if (lo != nullptr) lo[at] = pf_cast<T16>(v - Elem<T16>::to_f32(h));
 }
 
+// the same for N neighbouring values as 16-byte stores (N a multiple of 8, hi + at and lo + at on 16-byte boundaries)
+template <typename T16, int N> __device__ inline void pf_store_run(T16* hi, T16* lo, size_t at, const float (&v)[N]) {
+#pragma unroll
+    for (int i = 0; i < N; i += 8) {
+        uint32_t h[4], l[4];
+#pragma unroll
+        for (int k = 0; k < 4; ++k) {
+            const T16 a = pf_cast<T16>(v[i + 2 * k]), b = pf_cast<T16>(v[i + 2 * k + 1]);
+            const T16 c = pf_cast<T16>(v[i + 2 * k] - Elem<T16>::to_f32(a)), d = pf_cast<T16>(v[i + 2 * k + 1] - Elem<T16>::to_f32(b));
+            h[k] = (uint32_t)*reinterpret_cast<const unsigned short*>(&a) | (uint32_t)*reinterpret_cast<const unsigned short*>(&b) << 16;
+            l[k] = (uint32_t)*reinterpret_cast<const unsigned short*>(&c) | (uint32_t)*reinterpret_cast<const unsigned short*>(&d) << 16;
+        }
+        *reinterpret_cast<uint4*>(hi + at + i) = make_uint4(h[0], h[1], h[2], h[3]);
+        if (lo != nullptr) *reinterpret_cast<uint4*>(lo + at + i) = make_uint4(l[0], l[1], l[2], l[3]);
+    }
+}
+
 template <typename T16> struct PfEpiGate {  // columns (2j, 2j+1) = (w1, w3) column j: gate[j] = act(y1) * y3
     T16* gate;
     T16* gate_lo;
     int ld, act;
     __device__ void operator()(int, int row, int col, const float (&v)[32]) const {
         const size_t at = (size_t)row * ld + (col >> 1);
+        float g[16];
 #pragma unroll
         for (int j = 0; j < 16; ++j) {
             const float y1 = v[2 * j], y3 = v[2 * j + 1];
@@ -170,7 +188,13 @@ template <typename T16> struct PfEpiGate {  // columns (2j, 2j+1) = (w1, w3) col
             } else {
                 a = y1 / (1.0f + expf(-y1));
             }
-            pf_store(gate, gate_lo, at + j, a * y3);
+            g[j] = a * y3;
+        }
+        if (ld % 8 == 0) {
+            pf_store_run(gate, gate_lo, at, g);
+        } else {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) pf_store(gate, gate_lo, at + j, g[j]);
         }
     }
 };
