@@ -35,7 +35,7 @@ cudaError_t hybrid_step_t(cd_model* m, const cd_step& p) {
     const cd_config& c = m->cfg;
     cd_hybrid_state& S = *m->hybrid;
     const float mult = S.cfg.residual_mult, eps = S.cfg.eps;
-    const int D = c.dim;
+    const int D = c.dim, n = S.cfg.width;  // width padded to 8 with zeros, and the model's own
     cudaError_t e;
 #define TRY(x) do { e = (x); if (e != cudaSuccess) return e; } while (0)
     m->cur_cls = CLS_MISC;
@@ -54,8 +54,8 @@ cudaError_t hybrid_step_t(cd_model* m, const cd_step& p) {
     // the last sublayer's output, still to be normed and added: y, or two parallel mixers' outputs of layer `pair`
     struct { const float* y; VecNorm post; const cd_hybrid_layer* pair; } behind = {nullptr, {}, nullptr};
     float *yl = S.y, *yr = S.y + D;
-    auto residual = [&](const VecNorm& pre, const float* add = nullptr) { return InResidual{x[cur], behind.y, add, x[cur ^ 1], behind.post, pre, mult, eps, D}; };
-    auto mix_in = [&](const cd_hybrid_layer& L) { return InParallelMix{x[cur], yl, yr, L.out_l, L.out_r, L.post1.w, x[cur ^ 1], mult, eps, D}; };
+    auto residual = [&](const VecNorm& pre, const float* add = nullptr) { return InResidual{x[cur], behind.y, add, x[cur ^ 1], behind.post, pre, mult, eps, n}; };
+    auto mix_in = [&](const cd_hybrid_layer& L) { return InParallelMix{x[cur], yl, yr, L.out_l, L.out_r, L.post1.w, x[cur ^ 1], mult, eps, n}; };
     // the next GEMV's first rows, pulled into L2 behind a GEMV's own last loads
     auto hint = [&](const void* w, int K, int N, int unit) {
         m->next_stream = NextStream{m->prefetch_kb > 0 ? w : nullptr, Wfmt<WT>::row_stride(K), N / unit, unit, (uint32_t)m->prefetch_kb * 1024u};
@@ -126,7 +126,7 @@ cudaError_t hybrid_step_t(cd_model* m, const cd_step& p) {
             m->cur_cls = CLS_W13;
             int* sel = S.sel_ids + (size_t)S.runs[r].layer * SRC_MAX_LIST;
             TRY(launch_chain(m, moe_router_kernel<WT, RouterMixIn>, dim3((f.experts + 3) / 4), dim3(128), (size_t)std::max(D, f.experts + f.groups) * sizeof(float),
-                             RouterMixIn{x[cur], yl, yr, L.out_l, L.out_r, L.post1.w, x[cur ^ 1], mult, eps}, (const WT*)L.wr, S.router_logits, S.router_counter, sel,
+                             RouterMixIn{x[cur], yl, yr, L.out_l, L.out_r, L.post1.w, x[cur ^ 1], mult, eps, n}, (const WT*)L.wr, S.router_logits, S.router_counter, sel,
                              S.sel_w, S.loc_ids, S.loc_w, S.n_loc, D, RouteRule{f.experts, f.top, f.groups, f.keep}, 0, f.experts));
             cur ^= 1;
             const int units = f.top * L.ffp;
@@ -166,7 +166,8 @@ cudaError_t hybrid_step_t(cd_model* m, const cd_step& p) {
         InParallelMix in = mix_in(*behind.pair);
         in.x_out = m->x_a;
         TRY(launch_chain(m, vector_input_kernel<InParallelMix>, dim3(1), dim3(GEMV_CONSUMERS), 0, in, D));
-        return enqueue_head_t<WT, WT>(m, p, false, 0u, 0);
+        const InResidual head_in{m->x_a, nullptr, nullptr, m->x_b, VecNorm{}, S.final_norm, mult, eps, n};
+        return enqueue_head_t<WT, WT, InResidual>(m, p, false, 0u, 0, head_in);
     }
     if (p.head == HEAD_NONE) {
         InResidual in = residual(VecNorm{});
@@ -188,7 +189,7 @@ template <typename WT> cudaError_t hybrid_head_only_t(cd_model* m) {
     const cd_hybrid_state& S = *m->hybrid;
     m->cur_cls = CLS_HEAD;
     m->next_stream.w = nullptr;
-    const InResidual in{m->x_a, nullptr, nullptr, m->x_b, VecNorm{}, S.final_norm, 1.0f, S.cfg.eps, m->cfg.dim};
+    const InResidual in{m->x_a, nullptr, nullptr, m->x_b, VecNorm{}, S.final_norm, 1.0f, S.cfg.eps, S.cfg.width};
     return launch_gemv<WT, 1, false>(m, m->lm_head, m->x_a, nullptr, nullptr, m->v_loc, m->cfg.dim, EpiStore{m->logits}, SrcPlain{}, in);
 }
 cudaError_t hybrid_head_only(cd_model* m) { return m->opt.weight_dtype == CD_DTYPE_F32 ? hybrid_head_only_t<float>(m) : hybrid_head_only_t<__nv_bfloat16>(m); }
@@ -371,7 +372,7 @@ struct TensorSource {
 int check_limits(const HybridCfg& h, int dtype) {
     const int kmax = 8 * 256 * (dtype == CD_DTYPE_F32 ? 4 : 8);
     auto unsup = [&](const std::string& msg) { return fail(nullptr, CD_ERR_UNSUPPORTED, h.architecture + ": " + msg); };
-    if (h.width % 8 || h.width > kmax) return unsup("width must be a multiple of 8 and at most " + std::to_string(kmax));
+    if (h.width > kmax) return unsup("width is limited to " + std::to_string(kmax));
     if (h.side_dim > kmax) return unsup("token side wider than the GEMV tiling");
     for (const auto& L : h.layers) {
         if (L.has_attn() && (L.attn.dim > 256 || L.attn.vdim > 256)) return unsup("attention head widths are limited to 256");
@@ -430,6 +431,7 @@ int build(const std::string& json, const SafeTensors* file, size_t max_tokens, c
     AllocSpec spec;
     spec.family = &HYBRID_FAMILY;
     spec.local = cfg;
+    spec.local.dim = pad_to(h.width, 8);
     spec.local.nlayers = (int)runs.size();  // every pass through a layer has cache rows of its own
     for (const LayerRun& r : runs) spec.kv_row_elems.push_back(cached_elems(h.layers[r.layer]));
     cd_model* m = nullptr;
@@ -442,7 +444,7 @@ int build(const std::string& json, const SafeTensors* file, size_t max_tokens, c
     S->runs = runs;
     m->rms_eps = h.eps;
     m->needs_token = h.side_dim > 0;
-    const int D = h.width, nl = (int)h.layers.size();
+    const int width = h.width, D = pad_to(width, 8), nl = (int)h.layers.size();  // rows and vectors are padded with zeros
     const size_t es = esize(o.weight_dtype);
     const int epc = (int)(16 / es);
     S->layers.resize(nl);
@@ -596,16 +598,16 @@ int build(const std::string& json, const SafeTensors* file, size_t max_tokens, c
     T.file = file; T.seed = seed; T.std = std; T.m = m;
     auto load_norm = [&](const std::string& name, const VecNorm& v, bool around_zero) {
         if (!v.w) return;
-        T.vector(name, const_cast<float*>(v.w), D, around_zero ? 1.0f : 0.0f, around_zero ? 0.0f : 1.0f);
-        if (v.b) T.vector(name + ".b", const_cast<float*>(v.b), D, 0.0f, 0.0f);
+        T.vector(name, const_cast<float*>(v.w), width, around_zero ? 1.0f : 0.0f, around_zero ? 0.0f : 1.0f);
+        if (v.b) T.vector(name + ".b", const_cast<float*>(v.b), width, 0.0f, 0.0f);
     };
-    T.matrix("embed", m->embed, h.vocab, D, D);
-    if (!h.tied) T.matrix("head", m->lm_head, h.vocab, D, D);
+    T.matrix("embed", m->embed, h.vocab, width, D);
+    if (!h.tied) T.matrix("head", m->lm_head, h.vocab, width, D);
     load_norm("final.norm", S->final_norm, !h.layer_norm);
     if (h.side_dim) T.matrix("side.embed", S->side_embed, h.vocab, S->side_ld(), S->side_ld());
     if (h.loop_times) {
-        const std::vector<float> v = T.values("loop.step", {(size_t)h.loop_times, (size_t)D}, 0.0f);
-        T.upload("loop.step", S->loop_step, v.data(), v.size() * 4);
+        const std::vector<float> v = T.values("loop.step", {(size_t)h.loop_times, (size_t)width}, 0.0f);
+        for (int t = 0; t < h.loop_times; ++t) T.upload("loop.step", S->loop_step + (size_t)t * D, v.data() + (size_t)t * width, (size_t)width * 4);
     }
     for (int l = 0; l < nl && !T.rc; ++l) {
         cd_hybrid_layer& L = S->layers[l];
@@ -615,7 +617,7 @@ int build(const std::string& json, const SafeTensors* file, size_t max_tokens, c
         const FfnCfg& f = L.cfg.mlp;
         const bool pair = L.cfg.mixer == HybridLayerCfg::PARALLEL;
         const std::string p = "l" + std::to_string(l) + ".", pl = p + (pair ? "mix.left." : "mix."), pr = p + (pair ? "mix.right." : "mix."), pm = p + "mlp.";
-        auto rows = [&](const std::string& name, int first, int n) { T.matrix(name, (char*)L.wmix + (size_t)first * D * es, n, D, D); };
+        auto rows = [&](const std::string& name, int first, int n) { T.matrix(name, (char*)L.wmix + (size_t)first * D * es, n, width, D); };
         auto rotation = [&](const RotCfg& rot) {
             const std::vector<double> v = rot_frequencies(rot);
             if (!v.empty()) T.upload(p + "rotation", L.freq, v.data(), v.size() * sizeof(double));
@@ -623,7 +625,7 @@ int build(const std::string& json, const SafeTensors* file, size_t max_tokens, c
         if (L.cfg.has_attn()) {
             rows(pl + "q", L.proj.lq, a.heads * a.maps * a.dim); rows(pl + "k", L.proj.lk, a.kv_heads * a.maps * a.dim); rows(pl + "v", L.proj.lv, a.kv_heads * a.vdim);
             if (a.gate != AttnCfg::GATE_NONE) rows(pl + "g", L.proj.lg, a.gate == AttnCfg::GATE_HEAD ? a.heads : a.heads * a.vdim);
-            T.matrix(pl + "o", L.wo_l, D, a.heads * a.vdim, L.kl);
+            T.matrix(pl + "o", L.wo_l, width, a.heads * a.vdim, L.kl);
             if (a.qk_norm) { T.vector(pl + "q.norm", L.q_norm, a.heads * a.dim, 0.f, 1.f); T.vector(pl + "k.norm", L.k_norm, a.kv_heads * a.dim, 0.f, 1.f); }
             if (a.sink) T.vector(pl + "sink", L.sink, a.heads, 0.f, 0.f);
             if (a.distance_bias) {  // slopes 2^(-8 (h + 1) / H)
@@ -658,9 +660,9 @@ int build(const std::string& json, const SafeTensors* file, size_t max_tokens, c
                 T.upload(pr + "decay", L.log_decay, ld.data(), ld.size() * 4);
             }
             T.vector(pr + "norm", L.mem_norm, r.heads * r.vdim, 0.f, 1.f);
-            T.matrix(pr + "o", pair ? L.wo_r : L.wo_l, D, r.heads * r.vdim, pair ? L.kr : L.kl);
+            T.matrix(pr + "o", pair ? L.wo_r : L.wo_l, width, r.heads * r.vdim, pair ? L.kr : L.kl);
         }
-        if (pair) { T.vector(pl + "out", L.out_l, D, 0.f, 1.f); T.vector(pr + "out", L.out_r, D, 0.f, 1.f); }
+        if (pair) { T.vector(pl + "out", L.out_l, width, 0.f, 1.f); T.vector(pr + "out", L.out_r, width, 0.f, 1.f); }
         if (L.cfg.mixer == HybridLayerCfg::LATENT) {
             const int nq = t.heads * (t.dim + t.rot_dim), C = L.ld.latent;
             rows(pl + "q", 0, nq); rows(pl + "dkv", nq, t.rank + t.rot_dim);
@@ -676,14 +678,14 @@ int build(const std::string& json, const SafeTensors* file, size_t max_tokens, c
             }
             if (o.weight_dtype != CD_DTYPE_F32) T.matrix(pl + "uk", L.wukv, t.heads * t.dim, t.rank, C);
             T.matrix(pl + "uv", L.wuv, t.heads * t.vdim, t.rank, C);
-            T.matrix(pl + "o", L.wo_l, D, t.heads * t.vdim, L.kl);
+            T.matrix(pl + "o", L.wo_l, width, t.heads * t.vdim, L.kl);
         }
         // with norms ahead of the sublayers those are "norm1", "norm2" and the ones behind have a b; without, the plain names
         load_norm(p + "norm1", L.pre1, !h.layer_norm);
         load_norm(p + (h.pre_norms ? "norm1b" : "norm1"), L.post1, !h.layer_norm);
         if (h.side_dim) {
-            T.matrix(p + "side.gate", L.side_gate, h.side_dim, D, D);
-            T.matrix(p + "side.proj", L.side_proj, D, h.side_dim, S->side_pad());
+            T.matrix(p + "side.gate", L.side_gate, h.side_dim, width, D);
+            T.matrix(p + "side.proj", L.side_proj, width, h.side_dim, S->side_pad());
             load_norm(p + "side.norm", L.side_norm, false);
         }
         if (f.kind == FfnCfg::NONE) continue;
@@ -691,14 +693,14 @@ int build(const std::string& json, const SafeTensors* file, size_t max_tokens, c
         load_norm(p + (h.pre_norms ? "norm2b" : "norm2"), L.post2, !h.layer_norm);
         auto ffn = [&](const std::string& q, size_t i) {
             char* w13 = (char*)L.w13 + i * 2 * L.ffp * D * es;
-            T.matrix(q + "gate", w13, f.ff, D, D, 2, 0);
-            T.matrix(q + "up", w13, f.ff, D, D, 2, 1);
-            T.matrix(q + "down", (char*)L.w2 + i * D * L.ffp * es, D, f.ff, L.ffp);
+            T.matrix(q + "gate", w13, f.ff, width, D, 2, 0);
+            T.matrix(q + "up", w13, f.ff, width, D, 2, 1);
+            T.matrix(q + "down", (char*)L.w2 + i * D * L.ffp * es, width, f.ff, L.ffp);
         };
         if (f.kind == FfnCfg::DENSE) {
             ffn(pm, 0);
         } else {
-            T.matrix(pm + "router", L.wr, f.experts, D, D);
+            T.matrix(pm + "router", L.wr, f.experts, width, D);
             for (int i = 0; i < f.experts; ++i) ffn(pm + "e" + std::to_string(i) + ".", (size_t)i);
         }
     }

@@ -133,9 +133,9 @@ struct cd_hybrid_state {
     std::vector<cd::LayerRun> runs;
     std::vector<size_t> state_off;  // per run: its recurrent state inside a state slot (floats)
     cd::VecNorm final_norm{};
-    float* loop_step = nullptr;     // [loop_times][width]
+    float* loop_step = nullptr;     // [loop_times][width, padded]
     void* side_embed = nullptr;     // [vocab][layers * side_dim]
-    const float* step_vector(const cd::LayerRun& r) const { return r.step < 0 ? nullptr : loop_step + (size_t)r.step * cfg.width; }
+    const float* step_vector(const cd::LayerRun& r) const { return r.step < 0 ? nullptr : loop_step + (size_t)r.step * cd::pad_to(cfg.width, 8); }
     int side_ld() const { return (int)layers.size() * cfg.side_dim; }
     int side_pad() const { return cd::pad_to(cfg.side_dim, 8); }
     // recurrent state: slot 0 is the running sequence's, the others keep it at earlier lengths so that a session can

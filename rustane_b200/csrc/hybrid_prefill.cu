@@ -155,7 +155,7 @@ int ensure_workspace(cd_model* m, HybridPrefill* w, size_t n, size_t piece) {
 template <typename KT>
 int run_piece(cd_model* m, HybridPrefill* w, float* x, const uint32_t* ids, int rows, int pos0, bool split) {
     cd_hybrid_state& S = *m->hybrid;
-    const int D = m->cfg.dim, y_ld = (int)round_up(D, 32), side = S.cfg.side_dim, nruns = (int)S.runs.size();
+    const int D = m->cfg.dim, y_ld = (int)round_up(D, 32), side = S.cfg.side_dim, nruns = (int)S.runs.size(), width = S.cfg.width;
     const float mult = S.cfg.residual_mult, eps = S.cfg.eps;
     typedef __nv_bfloat16 AT;
     const size_t R = w->rows;
@@ -168,7 +168,7 @@ int run_piece(cd_model* m, HybridPrefill* w, float* x, const uint32_t* ids, int 
     };
     // residual stream behind y and the operand of the linear that follows: `pre` of it
     auto settle = [&](const char* what, const float* y, const VecNorm& post, const VecNorm& pre, const float* add = nullptr, const int* slots = nullptr, int top = 0) {
-        residual_rows_kernel<AT><<<rows, 256, D * 4, m->stream>>>(ResidualRows{x, y, y_ld, slots, w->sel_w, top, post, add, pre, mult, eps, D}, xn, xn_lo);
+        residual_rows_kernel<AT><<<rows, 256, D * 4, m->stream>>>(ResidualRows{x, y, y_ld, slots, w->sel_w, top, post, add, pre, mult, eps, width, D}, xn, xn_lo);
         check(what);
     };
     settle("embedding rows", nullptr, VecNorm{}, S.layers[S.runs[0].layer].pre1, S.step_vector(S.runs[0]));
@@ -242,7 +242,7 @@ int run_piece(cd_model* m, HybridPrefill* w, float* x, const uint32_t* ids, int 
             float *yl = w->y, *yr = w->y + R * (size_t)y_ld;
             gemm("attention output", attn, attn_lo, L.wo_l, rows, D, L.kl, D, PfEpiPartial{yl, y_ld});
             gemm("memory output", memn, memn_lo, L.wo_r, rows, D, L.kr, D, PfEpiPartial{yr, y_ld});
-            parallel_mix_rows_kernel<AT><<<rows, 256, D * 4, m->stream>>>(x, yl, yr, y_ld, L.out_l, L.out_r, L.post1.w, mult, eps, D, xn, xn_lo);
+            parallel_mix_rows_kernel<AT><<<rows, 256, D * 4, m->stream>>>(x, yl, yr, y_ld, L.out_l, L.out_r, L.post1.w, mult, eps, width, D, xn, xn_lo);
             check("residual behind the mixers");
         } else {
             const bool mem = L.cfg.mixer == HybridLayerCfg::MEMORY;

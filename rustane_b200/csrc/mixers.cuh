@@ -80,6 +80,7 @@ struct VecNorm {
 
 // ---------------------------------------------------------------------- inputs of the streamed GEMV (kernels.cuh, GemvIn)
 // x' = x + mult * post(y) + add, published; the GEMV's input is pre(x').  y (a sublayer's output) and add may be absent.
+// n: entries the norms are over; the vectors are padded with zeros behind them, weights and biases too.
 struct InResidual {
     static constexpr bool CUSTOM = true;
     const float *x, *y, *add;
@@ -105,7 +106,10 @@ struct InResidual {
         for (int i = 0; i < NITER; ++i) {
             if (tid + i * GEMV_CONSUMERS < nchunks) {
 #pragma unroll
-                for (int e = 0; e < EPC; ++e) { const float d = v[i][e] - mean; ss = fmaf(d, d, ss); }
+                for (int e = 0; e < EPC; ++e) {
+                    const float d = (tid + i * GEMV_CONSUMERS) * EPC + e < n ? v[i][e] - mean : 0.0f;
+                    ss = fmaf(d, d, ss);
+                }
             }
         }
         r = 1.0f / sqrtf(consumer_sum(ss, red, group) * inv_n + eps);

@@ -750,19 +750,19 @@ __global__ void __launch_bounds__(256) mem_rows_kernel(const float* __restrict__
 template <typename AT>
 __global__ void __launch_bounds__(256) parallel_mix_rows_kernel(float* __restrict__ x, const float* __restrict__ yl, const float* __restrict__ yr, int y_ld,
                                                                 const float* __restrict__ wl, const float* __restrict__ wr, const float* __restrict__ gain,
-                                                                float mult, float eps, int D, AT* __restrict__ hi, AT* __restrict__ lo) {
+                                                                float mult, float eps, int n, int D, AT* __restrict__ hi, AT* __restrict__ lo) {
     extern __shared__ float mixed[];  // [D]
     __shared__ float red[32];
     const float *a = yl + (size_t)blockIdx.x * y_ld, *b = yr + (size_t)blockIdx.x * y_ld;
     float sl = 0.0f, sr = 0.0f, ss = 0.0f;
     for (int i = threadIdx.x; i < D; i += 256) { sl = fmaf(a[i], a[i], sl); sr = fmaf(b[i], b[i], sr); }
-    const float rl = 0.5f / sqrtf(block_sum(sl, red) * (1.0f / (float)D) + eps), rr = 0.5f / sqrtf(block_sum(sr, red) * (1.0f / (float)D) + eps);
+    const float rl = 0.5f / sqrtf(block_sum(sl, red) * (1.0f / (float)n) + eps), rr = 0.5f / sqrtf(block_sum(sr, red) * (1.0f / (float)n) + eps);
     for (int i = threadIdx.x; i < D; i += 256) {
         const float z = a[i] * rl * wl[i] + b[i] * rr * wr[i];
         mixed[i] = z;
         ss = fmaf(z, z, ss);
     }
-    const float r = mult / sqrtf(block_sum(ss, red) * (1.0f / (float)D) + eps);
+    const float r = mult / sqrtf(block_sum(ss, red) * (1.0f / (float)n) + eps);
     for (int i = threadIdx.x; i < D; i += 256) {
         const size_t at = (size_t)blockIdx.x * D + i;
         const float v = x[at] + mixed[i] * r * gain[i];
@@ -771,17 +771,17 @@ __global__ void __launch_bounds__(256) parallel_mix_rows_kernel(float* __restric
     }
 }
 
-// mean and reciprocal deviation of a row in shared memory
-__device__ inline void row_moments(const float* row, int D, int kind, float eps, float* red, float& mean, float& r) {
+// mean and reciprocal deviation of the first n entries of a row in shared memory
+__device__ inline void row_moments(const float* row, int n, int kind, float eps, float* red, float& mean, float& r) {
     mean = 0.0f;
     if (kind == VecNorm::LAYER) {
         float s = 0.0f;
-        for (int i = threadIdx.x; i < D; i += 256) s += row[i];
-        mean = block_sum(s, red) * (1.0f / (float)D);
+        for (int i = threadIdx.x; i < n; i += 256) s += row[i];
+        mean = block_sum(s, red) * (1.0f / (float)n);
     }
     float ss = 0.0f;
-    for (int i = threadIdx.x; i < D; i += 256) { const float v = row[i] - mean; ss = fmaf(v, v, ss); }
-    r = 1.0f / sqrtf(block_sum(ss, red) * (1.0f / (float)D) + eps);
+    for (int i = threadIdx.x; i < n; i += 256) { const float v = row[i] - mean; ss = fmaf(v, v, ss); }
+    r = 1.0f / sqrtf(block_sum(ss, red) * (1.0f / (float)n) + eps);
 }
 
 // x += mult * post(y) + add, and pre(x) as a GEMM operand (InResidual, mixers.cuh).  y: none, one row per token, or (slots !=
@@ -797,7 +797,7 @@ struct ResidualRows {
     const float* add;
     VecNorm pre;
     float mult, eps;
-    int D;
+    int n, D;            // entries the norms are over; zeros follow up to D
 };
 template <typename AT>
 __global__ void __launch_bounds__(256) residual_rows_kernel(ResidualRows p, AT* __restrict__ hi, AT* __restrict__ lo) {
@@ -815,7 +815,7 @@ __global__ void __launch_bounds__(256) residual_rows_kernel(ResidualRows p, AT* 
             }
             sum[i] = v;
         }
-        if (normed) row_moments(sum, p.D, p.post.kind, p.eps, red, mean, r);
+        if (normed) row_moments(sum, p.n, p.post.kind, p.eps, red, mean, r);
     }
     r *= p.mult;
     for (int i = threadIdx.x; i < p.D; i += 256) {
@@ -828,7 +828,7 @@ __global__ void __launch_bounds__(256) residual_rows_kernel(ResidualRows p, AT* 
         sum[i] = v;
     }
     const bool ahead = p.pre.kind != VecNorm::NONE;
-    if (ahead) row_moments(sum, p.D, p.pre.kind, p.eps, red, mean, r);
+    if (ahead) row_moments(sum, p.n, p.pre.kind, p.eps, red, mean, r);
     for (int i = threadIdx.x; i < p.D; i += 256) {
         float v = sum[i];
         if (ahead) v = (v - mean) * r * p.pre.w[i] + (p.pre.b != nullptr ? p.pre.b[i] : 0.0f);

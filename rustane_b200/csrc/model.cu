@@ -414,11 +414,11 @@ int cd_decode_token(cd_model* m, const float* x_in, float* x_out) {
     if (int g_ = hidden_input_guard(m)) return g_;
     int rc = check_room(m, 1);
     if (rc) return rc;
-    CK(m, cudaMemcpyAsync(m->x_a, x_in, (size_t)m->cfg.dim * 4, cudaMemcpyHostToDevice, m->stream));
+    CK(m, cudaMemcpyAsync(m->x_a, x_in, (size_t)m->full_cfg.dim * 4, cudaMemcpyHostToDevice, m->stream));
     if ((rc = set_state(m, 0))) return rc;
     cd_step p{0, HEAD_NONE};
     if ((rc = run_step(m, p))) return rc;
-    CK(m, cudaMemcpyAsync(x_out, m->x_a, (size_t)m->cfg.dim * 4, cudaMemcpyDeviceToHost, m->stream));
+    CK(m, cudaMemcpyAsync(x_out, m->x_a, (size_t)m->full_cfg.dim * 4, cudaMemcpyDeviceToHost, m->stream));
     CK(m, cudaMemcpyAsync(&m->h_in[2], &m->st->error, 4, cudaMemcpyDeviceToHost, m->stream));
     CK(m, cudaStreamSynchronize(m->stream));
     if (m->h_in[2]) return device_wait_failed(m, (int)m->h_in[2], "");
@@ -435,7 +435,7 @@ int cd_decode_token_from_id(cd_model* m, uint32_t token, float* x_out) {
     if ((rc = set_state(m, token))) return rc;
     cd_step p{1, HEAD_NONE};
     if ((rc = run_step(m, p))) return rc;
-    CK(m, cudaMemcpyAsync(x_out, m->x_a, (size_t)m->cfg.dim * 4, cudaMemcpyDeviceToHost, m->stream));
+    CK(m, cudaMemcpyAsync(x_out, m->x_a, (size_t)m->full_cfg.dim * 4, cudaMemcpyDeviceToHost, m->stream));
     CK(m, cudaMemcpyAsync(&m->h_in[2], &m->st->error, 4, cudaMemcpyDeviceToHost, m->stream));
     CK(m, cudaStreamSynchronize(m->stream));
     if (m->h_in[2]) return device_wait_failed(m, (int)m->h_in[2], "");
@@ -462,7 +462,7 @@ int cd_decode_token_argmax(cd_model* m, const float* x_in, uint32_t* out) {
     if (int g_ = hidden_input_guard(m)) return g_;
     int rc = check_room(m, 1);
     if (rc) return rc;
-    CK(m, cudaMemcpyAsync(m->x_a, x_in, (size_t)m->cfg.dim * 4, cudaMemcpyHostToDevice, m->stream));
+    CK(m, cudaMemcpyAsync(m->x_a, x_in, (size_t)m->full_cfg.dim * 4, cudaMemcpyHostToDevice, m->stream));
     return argmax_common(m, 0, 0, out);
 }
 

@@ -349,7 +349,7 @@ mla_out_kernel(const float* __restrict__ part_acc, const float* __restrict__ par
                const DevState* st, MlaDims d, int nsplit_max, int tile) {
     extern __shared__ float sm[];  // [C] the head's latent-space output, then [nsplit] slice weights
     constexpr float NEG = -3.402823466e+38f;
-    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nw = blockDim.x >> 5;
+    const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;  // eight warps
     const int H = d.heads, C = d.latent, V = d.vdim, h = blockIdx.x;
     float* lat = sm;
     float* wsl = sm + C;
@@ -396,12 +396,12 @@ mla_out_kernel(const float* __restrict__ part_acc, const float* __restrict__ par
     __syncthreads();
     // this CTA's 32 output rows of the head: four rows per warp, their loads in flight together
     const int dv0 = blockIdx.y * 32 + warp * 4;
-    if (nw == 8 && dv0 + 4 <= V) {
+    if (dv0 + 4 <= V) {
         float y[4];
         warp_rows_dot<WT, 4>(wuv_t + ((size_t)h * V + dv0) * C, (size_t)C, lat, C, lane, y);
         if (lane < 4) attn_out[(size_t)h * V + dv0 + lane] = lane == 0 ? y[0] : lane == 1 ? y[1] : lane == 2 ? y[2] : y[3];
     } else {
-        for (int dv = blockIdx.y * 32 + warp; dv < min(V, (int)blockIdx.y * 32 + 32); dv += nw) {
+        for (int dv = dv0; dv < V; ++dv) {
             const float v = warp_row_dot<WT>(wuv_t + ((size_t)h * V + dv) * C, lat, C, lane);
             if (lane == 0) attn_out[(size_t)h * V + dv] = v;
         }
@@ -695,6 +695,7 @@ struct RouterMixIn {  // the residual stream behind two parallel mixers (InParal
     const float *x, *yl, *yr, *wl, *wr, *gain;
     float* out;
     float mult, eps;
+    int n;               // entries the norms are over (zeros behind them)
     __device__ float fill(float* xs, float* red, int dim, bool writer) const {  // dim is a multiple of 4
         const int n4 = dim / 4, step = blockDim.x;
         auto at = [](const float* p, int i) { return __ldcg(reinterpret_cast<const float4*>(p) + i); };
@@ -707,8 +708,8 @@ struct RouterMixIn {  // the residual stream behind two parallel mixers (InParal
             sl += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
             sr += b.x * b.x + b.y * b.y + b.z * b.z + b.w * b.w;
         }
-        const float rl = 0.5f / sqrtf(block_sum(sl, red) * (1.0f / (float)dim) + eps);
-        const float rr = 0.5f / sqrtf(block_sum(sr, red) * (1.0f / (float)dim) + eps);
+        const float rl = 0.5f / sqrtf(block_sum(sl, red) * (1.0f / (float)n) + eps);
+        const float rr = 0.5f / sqrtf(block_sum(sr, red) * (1.0f / (float)n) + eps);
 #pragma unroll 4
         for (int i = threadIdx.x; i < n4; i += step) {
             const float4 a = at(yl, i), b = at(yr, i), p = weight(wl, i), q = weight(wr, i);
@@ -716,7 +717,7 @@ struct RouterMixIn {  // the residual stream behind two parallel mixers (InParal
             x4[i] = z;
             ss += z.x * z.x + z.y * z.y + z.z * z.z + z.w * z.w;
         }
-        const float r = mult / sqrtf(block_sum(ss, red) * (1.0f / (float)dim) + eps);
+        const float r = mult / sqrtf(block_sum(ss, red) * (1.0f / (float)n) + eps);
 #pragma unroll 4
         for (int i = threadIdx.x; i < n4; i += step) {
             const float4 b = at(x, i), g = weight(gain, i), z = x4[i];

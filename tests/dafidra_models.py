@@ -185,3 +185,8 @@ NARROW = config(72, 57, [                                 # widths that are no m
     (attn(3, 3, 12, 4, 6, 0.6, 0.2, 2), memory(3, 6, 10, 7.0), moe(40, 6, 12, (10, 7))),
     (attn(4, 1, 20, 28, 150, 0.25), memory(1, 4, 100, 7.0), dense(20)),
 ], eps=1e-4, mult=0.6)
+RAGGED = config(61, 75, [                                 # a width that fits no chunk
+    (attn(3, 1, 12, 10, 9, 0.5, 0.2, 4), memory(2, 9, 7, 7.0), moe(6, 2, 11)),
+    (attn(2, 2, 20, 6, None, 0.25), memory(3, 5, 12, 9.0), dense(19)),
+    (attn(1, 1, 8, 8, 5, 0.4), memory(1, 4, 4, 7.0), None),
+], eps=1e-4, mult=0.8)

@@ -175,3 +175,8 @@ TAIL = config(72, 57, [                                   # the loop ends ahead 
     (diff(3, 3, 20, 28, 0.25, rot(4, 100.0)), 24),
     (lightning(5, 6, 10, (0.99, 0.9, 0.5, 0.999, 0.1)), None),
 ], loop=(1, 2, 1), side=1, eps=1e-4)
+RAGGED = config(91, 75, [                                 # a width that fits no chunk
+    (diff(2, 1, 10, 14, 0.3, rot(6, 200.0)), 17),
+    (latent(3, 9, 2, 11, 21, 7, 0.3), None),
+    (lightning(3, 7, 5, (0.9, 0.6, 0.97)), 23),
+], loop=(0, 2, 2), side=3)

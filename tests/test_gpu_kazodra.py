@@ -18,7 +18,7 @@ ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 # distance to an oracle whose cache rounds its rows the same way.
 TOL = {"f32": 4e-5, "bf16": 1.5e-2}
 KEPT = {"decoded": 1e-3, "prompt": 6e-3}   # a prompt rounds the expanded keys and values of latent attention once more
-SEED = {"ODD": 2, "WIDE": 5, "BROAD": 1, "PLAIN": 1, "TAIL": 3}
+SEED = {"ODD": 2, "WIDE": 5, "BROAD": 1, "PLAIN": 1, "TAIL": 3, "RAGGED": 4}
 
 
 @pytest.fixture(scope="module")
@@ -76,6 +76,7 @@ def test_whole_prompt_and_decoding_match_the_oracle(R, made, name, dtype):
 
 @pytest.mark.parametrize("name,portions", [
     ("ODD", [2] * 100), ("ODD", [9, 2, 13, 8, 64, 3, 65, 2, 34]), ("WIDE", [63, 2, 64, 1, 65, 5]), ("PLAIN", [8] * 25), ("BROAD", [130, 3, 50, 2, 15]), ("TAIL", [2, 11, 100, 1, 86]),
+    ("RAGGED", [50, 2, 9, 1, 138]),
 ])
 def test_portions_of_a_prompt_do_not_change_its_logits(R, made, name, portions):
     cfg, _, path, ids, ref = made(name)
