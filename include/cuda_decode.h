@@ -223,7 +223,11 @@ int cd_moe_last_experts(cd_model* m, int layer, int32_t* out_ids, size_t cap);
  * model.safetensors (no counterpart in the reference, whose one architecture is fixed by its checkpoint header).
  * Registered: "Dafidra" - per layer a windowed softmax attention (whole-projection q/k norm, query temperature, linear
  * distance bias, sink, per-head output gate) and a matrix memory (mLSTM) side by side on the un-normed residual stream,
- * norms on the sublayers' outputs, then a dense or a routed feed-forward.
+ * norms on the sublayers' outputs, then a dense or a routed feed-forward.  "Kazodra" - per layer latent attention over a
+ * window, linear attention with constant decays or differential attention, then a dense feed-forward, layer norms ahead of
+ * and behind each, and a gated part of a second embedding of the token; a run of layers may be passed several times.  Its
+ * layers read the token id, so cd_decode_token and cd_decode_token_argmax (a hidden state as input) return
+ * CD_ERR_UNSUPPORTED where it has that embedding.
  * opts->weight_dtype: CD_DTYPE_BF16 (also for < 0) or CD_DTYPE_F32; one GPU.  max_tokens (0: 4096) bounds the sequence:
  * it becomes cd_config.seq.  Every call that takes a cd_model works on the handle except cd_seed_layer_cache_cf and
  * cd_decode_steps_samples (CD_ERR_UNSUPPORTED; the session then runs the samples one after the other).
